@@ -839,6 +839,66 @@ int b200_moe_route_grouped(const void* h, int64_t ldh, const float* wr, const fl
                            int W, int top, int n_groups, int keep, int* ids, float* wts, int T,
                            int dtype, void* stream);
 
+/* ---- parallel blocks with input convolutions and differential attention ---------------------------
+ * b200_gemm_16bit with out = xielu(result): z > 0: act_pos z^2 + z / 2; z <= 0: act_neg (e^z - 1 - z) + z / 2. */
+int b200_gemm_16bit_xielu(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* bias,
+                          void* out, int64_t ldc, int M, int N, int K, float act_pos, float act_neg,
+                          int dtype, void* stream);
+/* The same activation on rows [T, D]; out may be a column slice of wider rows.                       */
+int b200_xielu_rows(const void* z, int64_t ldz, void* out, int64_t ldo, int T, int D, float pos,
+                    float neg, int dtype, void* stream);
+/* y = x + a + b (fp32 residual x, terms optional) -> x_out (not x); r = 1 / sqrt(mean(y^2) + eps);
+ * h = y r w1;  out1 = h + causal convolution of h over the entry's tokens (cw [taps, W] fp32, row j times
+ * the h taps-1-j tokens back; cw NULL and taps 1: out1 = h);  out2 (optional) = y r w2.  state
+ * [slots, ld_state] fp32 keeps each sequence's last taps-1 h ([taps-1, W], oldest first), read at the start
+ * of a portion (zeros at position 0) and replaced at its end.  taps <= 16.                            */
+int b200_residual_norm_conv(const float* x, int64_t ldx, const void* a, int64_t lda, const void* b,
+                            int64_t ldb, float* x_out, int64_t ldxo, const float* w1, const float* w2,
+                            float eps, const float* cw, int taps, float* state, int64_t ld_state,
+                            const int64_t* slot, const int* tok_pos, const int* ext_start,
+                            const int* ext_len, void* out1, int64_t ld1, void* out2, int64_t ld2, int bs,
+                            int max_ext, int W, int dtype, void* stream);
+/* Projections y [T, (q_maps + k_maps) * D + v_channels] -> causal convolution per channel (cw
+ * [taps, channels] fp32, state as above over these channels; cw NULL: none) -> rotation of the first
+ * rot_dims coordinates of every query / key map in the half pairing -> q rows (fp32 and / or 16-bit),
+ * k and v into the token's pool row at k_off / v_off.  k_maps = v_channels = 0: queries only.        */
+int b200_conv_rot_write(const void* y, int64_t ldy, const float* cw, int taps, float* state,
+                        int64_t ld_state, const int64_t* slot, const int* tok_pos, const int* ext_start,
+                        const int* ext_len, const float* freq_hi, const float* freq_lo, int rot_dims,
+                        const int64_t* loc, void* pool, int64_t ld_pool, int k_off, int v_off, float* q32,
+                        int64_t ldq32, void* q16, int64_t ldq16, int q_maps, int k_maps, int D,
+                        int v_channels, int bs, int max_ext, int dtype, void* stream);
+/* Differential attention: per query head two maps q [H][2][D], per key/value head two key maps [2][D]
+ * (pool row at k_off + g * 2 * D) and one value [E] (at v_off + g * E); a_m = softmax(scale q_m k_m) v,
+ * d = a_1 - *lambda a_2, out[t, h * E ..] = d / sqrt(mean(d^2) + eps) * out_mult.  Position i sees
+ * floor(i / chunk) * chunk <= j <= i (chunk > 0), i - window < j <= i (window > 0), or all j <= i.
+ * tok_list (NULL: rows 0 .. rows-1) names the token rows.  CUDA cores, fp32 queries, E <= 256.        */
+int b200_diff_attn(const float* q, int64_t ldq, const void* pool, int64_t ld_pool, int k_off, int v_off,
+                   const int* req_to_token, int64_t ld_r2t, const int64_t* req_idx, const int* tok_pos,
+                   const int* tok_b, const int* tok_list, const float* lambda, float out_mult, float eps,
+                   float scale, int window, int chunk, void* out, int64_t ldo, int rows, int H, int G,
+                   int D, int E, int max_keys, int dtype, void* stream);
+/* The same with 16-bit queries on mma.sync, split over the keys; part_o fp32 [rows, H, 2, num_splits, E]
+ * and part_lse [rows, H, 2, num_splits] when num_splits > 1.  2D x E in {64, 128} x {64, 128}, 256 x 128. */
+int b200_diff_attn_mma_supported(int D, int E);
+int b200_diff_attn_mma_splits(int rows, int H, int G, int max_keys, int num_sms);
+int b200_diff_attn_mma(const void* q, int64_t ldq, const void* pool, int64_t ld_pool, int k_off, int v_off,
+                       const int* req_to_token, int64_t ld_r2t, const int64_t* req_idx,
+                       const int* tok_pos, const int* tok_b, const int* tok_list, const float* lambda,
+                       float out_mult, float eps, float scale, int window, int chunk, void* out,
+                       int64_t ldo, int rows, int H, int G, int D, int E, int num_splits, float* part_o,
+                       float* part_lse, int dtype, void* stream);
+/* The same for prompt portions on tcgen05 (batch entries as b200_attn_extend); sizes as above.  A
+ * bounded wait inside the kernel that runs out is reported by the error word (read and cleared by
+ * b200_diff_attn_extend_error) and by the next launch.                                               */
+int b200_diff_attn_extend_error(void);
+int b200_diff_attn_extend(const void* q, int64_t q_stride, const void* pool, int64_t ld_pool, int k_off,
+                          int v_off, void* o, int64_t o_stride, const int* req_to_token,
+                          int64_t rtt_stride, const int64_t* req_pool_indices, const int* prefix_lens,
+                          const int* extend_lens, const int* extend_start, int bs, int max_ext, int H,
+                          int G, int D, int E, float scale, int window, int chunk, const float* lambda,
+                          float out_mult, float eps, int dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -282,6 +282,33 @@ _SIGNATURES = {
                                         c_void_p]),
     "b200_moe_route_grouped": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                        c_int, c_void_p, c_void_p, c_int, c_int, c_void_p]),
+    "b200_gemm_16bit_xielu": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64,
+                                      c_int, c_int, c_int, c_float, c_float, c_int, c_void_p]),
+    "b200_xielu_rows": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_float, c_float, c_int,
+                                c_void_p]),
+    "b200_residual_norm_conv": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                                        c_int64, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p,
+                                        c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64,
+                                        c_void_p, c_int64, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_conv_rot_write": (c_int, [c_void_p, c_int64, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p,
+                                    c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                                    c_int64, c_int, c_int, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int,
+                                    c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_diff_attn": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_int64,
+                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_float,
+                               c_int, c_int, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
+                               c_int, c_void_p]),
+    "b200_diff_attn_mma_supported": (c_int, [c_int, c_int]),
+    "b200_diff_attn_mma_splits": (c_int, [c_int, c_int, c_int, c_int, c_int]),
+    "b200_diff_attn_mma": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_int64,
+                                   c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float,
+                                   c_float, c_int, c_int, c_void_p, c_int64, c_int, c_int, c_int, c_int,
+                                   c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]),
+    "b200_diff_attn_extend_error": (c_int, []),
+    "b200_diff_attn_extend": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_int64,
+                                      c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                      c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_float,
+                                      c_float, c_int, c_void_p]),
 }
 
 

@@ -12,6 +12,7 @@
 #pragma once
 #include <type_traits>
 
+#include "activation.cuh"
 #include "tc_common.cuh"
 
 namespace b200 {
@@ -34,6 +35,8 @@ struct GemmEpilogueParams {
   // on that share.  splits == 1: plain persistent path.
   int splits = 1;
   int kb_per_split = 0;
+  // ACT instances: out = xielu(result; act_pos, act_neg) before the store (activation.cuh)
+  float act_pos = 0.f, act_neg = 0.f;
 };
 
 template <int KIND>
@@ -119,7 +122,7 @@ __device__ __forceinline__ uint32_t pack_out2<__half>(float a, float b) {
 // ingest from 48 KiB to 32 KiB per K block (the measured limiter of the 128x256 tile).  A stage
 // may be refilled only when BOTH CTAs' MMAs have consumed it: tcgen05.commit multicasts its arrive
 // to both empty barriers (count 2).  tmap_b then describes BLOCK_N/2-row boxes.
-template <int KIND, int BLOCK_N, int STAGES, typename OutT, bool MC = false>
+template <int KIND, int BLOCK_N, int STAGES, typename OutT, bool MC = false, bool ACT = false>
 __global__ void __launch_bounds__(192, 1)
 gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b,
                const GemmEpilogueParams ep) {
@@ -287,6 +290,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
     const int quarter = warp & 3;  // TMEM lane quarter this warp may access
     OutT* out = static_cast<OutT*>(ep.out);
     const OutT* bias = static_cast<const OutT*>(ep.bias);
+    auto finish = [&](float v) { return ACT ? xielu_fast(v, ep.act_pos, ep.act_neg) : v; };
     int local = 0;
     for (int item = item0; item < num_items; item += item_step, ++local) {
       const int tile = MC ? item : item / S, ks = MC ? 0 : item - tile * S;
@@ -354,7 +358,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
               for (int e = 0; e < 4; ++e) {
                 const float s0 = sa * sbt[g * 8 + 2 * e], s1 = sa * sbt[g * 8 + 2 * e + 1];
                 const float b0 = bst[g * 8 + 2 * e], b1 = bst[g * 8 + 2 * e + 1];
-                packed[e] = pack_out2<OutT>(fmaf(sum[2 * e], s0, b0), fmaf(sum[2 * e + 1], s1, b1));
+                packed[e] = pack_out2<OutT>(finish(fmaf(sum[2 * e], s0, b0)), finish(fmaf(sum[2 * e + 1], s1, b1)));
               }
               *reinterpret_cast<uint4*>(orow + col0) =
                   make_uint4(packed[0], packed[1], packed[2], packed[3]);
@@ -364,7 +368,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
                 if (col0 + j >= ep.N) break;
                 const float sc = sa * sbt[g * 8 + j];
                 const float bb = bst[g * 8 + j];
-                orow[col0 + j] = from_float<OutT>(fmaf(sum[j], sc, bb));
+                orow[col0 + j] = from_float<OutT>(finish(fmaf(sum[j], sc, bb)));
               }
             }
           }
@@ -392,7 +396,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
                 float x0 = __uint_as_float(r[j]), x1 = __uint_as_float(r[j + 1]);
                 const float s0 = sa * sbt[c * 32 + j], s1 = sa * sbt[c * 32 + j + 1];
                 const float b0 = bst[c * 32 + j], b1 = bst[c * 32 + j + 1];
-                packed[e] = pack_out2<OutT>(fmaf(x0, s0, b0), fmaf(x1, s1, b1));
+                packed[e] = pack_out2<OutT>(finish(fmaf(x0, s0, b0)), finish(fmaf(x1, s1, b1)));
               }
               *reinterpret_cast<uint4*>(orow + col0 + v * 8) =
                   make_uint4(packed[0], packed[1], packed[2], packed[3]);
@@ -403,7 +407,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
               if (col0 + j >= ep.N) break;
               const float s = sa * sbt[c * 32 + j];
               const float b = bst[c * 32 + j];
-              orow[col0 + j] = from_float<OutT>(fmaf(__uint_as_float(r[j]), s, b));
+              orow[col0 + j] = from_float<OutT>(finish(fmaf(__uint_as_float(r[j]), s, b)));
             }
           }
         }
@@ -432,7 +436,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
 int splitk_pick(int tiles, int num_kb, int sms);
 
 // Host launcher: builds the two TMA descriptors and launches one CTA per SM (or per tile).
-template <int KIND, int BLOCK_N, int STAGES, typename OutT, bool MC = false>
+template <int KIND, int BLOCK_N, int STAGES, typename OutT, bool MC = false, bool ACT = false>
 int launch_gemm_tn(const void* a, int64_t lda, const void* b, int64_t ldb,
                    const GemmEpilogueParams& ep_in, cudaStream_t st, const char* timer_name,
                    bool allow_split = false) {
@@ -443,7 +447,7 @@ int launch_gemm_tn(const void* a, int64_t lda, const void* b, int64_t ldb,
   if (rc) return rc;
   rc = make_tmap_2d(&tb, b, ep.N, ep.K, ldb * C::ELT, MC ? BLOCK_N / 2 : BLOCK_N, C::BLOCK_K, C::ELT, true);
   if (rc) return rc;
-  auto kern = gemm_tn_kernel<KIND, BLOCK_N, STAGES, OutT, MC>;
+  auto kern = gemm_tn_kernel<KIND, BLOCK_N, STAGES, OutT, MC, ACT>;
   static bool attr_done = false;
   if (!attr_done) {
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,

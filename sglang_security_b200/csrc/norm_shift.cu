@@ -22,6 +22,9 @@
 //                          written (a model's final layer norm).
 //   act_and_mul_clamped  : out = g * sigmoid(slope * g) * (u + 1), g = min(z[:, :d], limit),
 //                          u = clamp(z[:, d:], -limit, limit)
+//   xielu_rows           : out = xielu(z; pos, neg) (activation.cuh); the result may be a column slice of
+//                          wider rows
+#include "activation.cuh"
 #include "common.cuh"
 
 namespace b200 {
@@ -139,6 +142,15 @@ act_and_mul_kernel(const T* __restrict__ z, int64_t ldz, T* __restrict__ out, in
     const float a = to_float<T>(from_float<T>(act_apply(to_float<T>(z[t * ldz + d]), kind)));
     out[t * ldo + d] = from_float<T>(a * to_float<T>(z[t * ldz + D + d]));
   }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads)
+xielu_rows_kernel(const T* __restrict__ z, int64_t ldz, T* __restrict__ out, int64_t ldo, int D, float pos,
+                  float neg) {
+  const int t = blockIdx.x;
+  for (int d = threadIdx.x; d < D; d += kRowThreads)
+    out[t * ldo + d] = from_float<T>(xielu_exact(to_float<T>(z[t * ldz + d]), pos, neg));
 }
 
 template <typename TA>
@@ -415,5 +427,24 @@ extern "C" int b200_act_and_mul_clamped(const void* z, int64_t ldz, void* out, i
   else B200_REQUIRE(false, "b200_act_and_mul_clamped: dtype %d", dtype);
 #undef LAUNCH
   B200_CHECK_LAUNCH("act_and_mul_clamped_kernel");
+  return 0;
+}
+
+extern "C" int b200_xielu_rows(const void* z, int64_t ldz, void* out, int64_t ldo, int T, int D, float pos,
+                               float neg, int dtype, void* stream) {
+  using namespace b200;
+  if (T == 0 || D == 0) return 0;
+  B200_REQUIRE(z && out && T > 0 && D > 0, "b200_xielu_rows: bad arguments");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  ScopedKernelTimer timer("xielu_rows", st);
+#define LAUNCH(TT)                                                                                   \
+  launch_kernel(xielu_rows_kernel<TT>, dim3(T), dim3(kRowThreads), 0, st, 1, 0,                      \
+                static_cast<const TT*>(z), ldz, static_cast<TT*>(out), ldo, D, pos, neg)
+  if (dtype == B200_BF16) LAUNCH(__nv_bfloat16);
+  else if (dtype == B200_F16) LAUNCH(__half);
+  else if (dtype == B200_F32) LAUNCH(float);
+  else B200_REQUIRE(false, "b200_xielu_rows: dtype %d", dtype);
+#undef LAUNCH
+  B200_CHECK_LAUNCH("xielu_rows_kernel");
   return 0;
 }
