@@ -633,12 +633,13 @@ extern "C" int b200_diff_attn_mma_supported(int D, int E) {
   return (dk == 64 && (E == 64 || E == 128)) || (dk == 128 && (E == 64 || E == 128)) || (dk == 256 && E == 128);
 }
 
-// CTAs that fill the machine twice over, never fewer than 4 tiles of work per CTA
+// As many splits as keep all CTAs resident at once (two per SM: a second, partly filled wave costs more than
+// longer parts), never fewer than 4 tiles of work per warp and part
 extern "C" int b200_diff_attn_mma_splits(int rows, int H, int G, int max_keys, int num_sms) {
   using namespace b200;
   if (rows <= 0 || G <= 0 || H <= 0 || max_keys <= 0) return 1;
   const int64_t base = static_cast<int64_t>(rows) * G * ceil_div(H / G, 8);
-  int64_t s = (2 * static_cast<int64_t>(num_sms) + base - 1) / base;
+  int64_t s = 2 * static_cast<int64_t>(num_sms) / base;
   const int64_t most = ceil_div(max_keys, 4 * kDiffAlign);
   s = s < most ? s : most;
   return static_cast<int>(s < 1 ? 1 : (s > 64 ? 64 : s));

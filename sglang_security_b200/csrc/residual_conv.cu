@@ -17,6 +17,8 @@
 //                        pairing: coordinate i with i + rot/2 of every head map) by position x frequency;
 //                        q out as fp32 and / or 16-bit rows, k and v into the token's pool row.
 // Norms, convolutions, angles and rotation are fp32.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace b200 {
@@ -39,6 +41,14 @@ __device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC]) {
     for (int e = 0; e < VEC; ++e) v[e] = to_float<T>(p[e]);
   }
 }
+
+// A piece as it lies in memory, for loads that are requested rows ahead of their use
+template <typename T, int VEC>
+struct Piece {
+  typename std::conditional<VEC == 4, typename std::conditional<sizeof(T) == 2, uint2, float4>::type, T>::type raw;
+  __device__ __forceinline__ void load(const T* p) { raw = *reinterpret_cast<const decltype(raw)*>(p); }
+  __device__ __forceinline__ void get(float (&v)[VEC]) const { load_vec<T, VEC>(reinterpret_cast<const T*>(&raw), v); }
+};
 
 template <typename T, int VEC>
 __device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
@@ -230,22 +240,49 @@ residual_norm_conv_kernel(const NormConvArgs p) {
       normed(q, v, h);
       hist.push(h);
     }
-#pragma unroll 4
-    for (int q = halo; q < halo + m; ++q) {
-      float v[VEC], h[VEC], y[VEC];
-      normed(q, v, h);
-      const int64_t row = r0 + i0 + (q - halo);
-      convolve<MT, VEC>(wk, h, hist, y);
+    // rows in batches: all loads of a batch are requested before its first row is used and stored
+    constexpr int RB = MT <= 4 ? 4 : 1;
+    for (int q0 = halo; q0 < halo + m; q0 += RB) {
+      Piece<float, VEC> px[RB];
+      Piece<T, VEC> ta[RB], tb[RB];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) y[e] += h[e];
-      hist.push(h);
-      store_vec<float, VEC>(p.x_out + row * p.ldxo + c, v);
-      store_vec<T, VEC>(o1 + row * p.ld1 + c, y);
-      if (o2) {
+      for (int i = 0; i < RB; ++i) {
+        const int64_t row = r0 + i0 + min(q0 + i - halo, m - 1);
+        px[i].load(p.x + row * p.ldx + c);
+        if (pa) ta[i].load(pa + row * p.lda + c);
+        if (pb) tb[i].load(pb + row * p.ldb + c);
+      }
+#pragma unroll
+      for (int i = 0; i < RB; ++i) {
+        const int q = q0 + i;
+        if (q >= halo + m) break;
+        const int64_t row = r0 + i0 + (q - halo);
         const float r = inv_s[q];
+        float v[VEC], h[VEC], y[VEC];
+        px[i].get(v);
+        if (pa) {
+          ta[i].get(h);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) y[e] = v[e] * r * w2[e];
-        store_vec<T, VEC>(o2 + row * p.ld2 + c, y);
+          for (int e = 0; e < VEC; ++e) v[e] += h[e];
+        }
+        if (pb) {
+          tb[i].get(h);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[e] += h[e];
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) h[e] = v[e] * r * w1[e];
+        convolve<MT, VEC>(wk, h, hist, y);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] += h[e];
+        hist.push(h);
+        store_vec<float, VEC>(p.x_out + row * p.ldxo + c, v);
+        store_vec<T, VEC>(o1 + row * p.ld1 + c, y);
+        if (o2) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) y[e] = v[e] * r * w2[e];
+          store_vec<T, VEC>(o2 + row * p.ld2 + c, y);
+        }
       }
     }
     if (first && st) {
@@ -366,35 +403,51 @@ conv_rot_write_kernel(const ConvRotArgs p) {
       store_vec<T, VEC>(pool + prow * p.ld_pool + (c < ck ? p.k_off + c - cq : p.v_off + c - ck), v);
     }
   };
-#pragma unroll 4
-  for (int q = 0; q < m; ++q) {
-    const int64_t row = r0 + i0 + q;
-    float va[VEC], vb[VEC], ya[VEC], yb[VEC];
-    load_vec<T, VEC>(yin + row * p.ldy + ca, va);
-    load_vec<T, VEC>(yin + row * p.ldy + cb, vb);
-    const int64_t prow = ca >= cq ? p.loc[row] : 0;
-    if (p.cw) {
-      convolve<MT, VEC>(wa, va, ha, ya);
-      convolve<MT, VEC>(wb, vb, hb, yb);
-      ha.push(va);
-      hb.push(vb);
-    } else {
+  constexpr int RB = MT <= 4 ? 4 : 1;                       // rows requested together
+  for (int q0 = 0; q0 < m; q0 += RB) {
+    Piece<T, VEC> pa[RB], pb[RB];
+    int64_t prow[RB];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        ya[e] = va[e];
-        yb[e] = vb[e];
-      }
+    for (int i = 0; i < RB; ++i) {
+      const int64_t row = r0 + i0 + min(q0 + i, m - 1);
+      pa[i].load(yin + row * p.ldy + ca);
+      pb[i].load(yin + row * p.ldy + cb);
+      prow[i] = ca >= cq ? p.loc[row] : 0;
     }
-    if (rotated) {
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        const float c = cs[q * half + f0 + e], s = sn[q * half + f0 + e], u = ya[e], v = yb[e];
-        ya[e] = fmaf(u, c, -v * s);
-        yb[e] = fmaf(v, c, u * s);
+    for (int i = 0; i < RB; ++i) {
+      const int q = q0 + i;
+      if (q >= m) break;
+      const int64_t row = r0 + i0 + q;
+      float va[VEC], vb[VEC], ya[VEC], yb[VEC];
+      pa[i].get(va);
+      pb[i].get(vb);
+      if (p.cw) {
+        convolve<MT, VEC>(wa, va, ha, ya);
+        convolve<MT, VEC>(wb, vb, hb, yb);
+        ha.push(va);
+        hb.push(vb);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          ya[e] = va[e];
+          yb[e] = vb[e];
+        }
       }
+      if (rotated) {
+        float c[VEC], s[VEC];
+        load_vec<float, VEC>(cs + q * half + f0, c);
+        load_vec<float, VEC>(sn + q * half + f0, s);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const float u = ya[e], v = yb[e];
+          ya[e] = fmaf(u, c[e], -v * s[e]);
+          yb[e] = fmaf(v, c[e], u * s[e]);
+        }
+      }
+      put(row, prow[i], ca, ya);
+      if (live_b) put(row, prow[i], cb, yb);
     }
-    put(row, prow, ca, ya);
-    if (live_b) put(row, prow, cb, yb);
   }
   if (first && st) {
     if (n > kConvTile) {                                    // the portion goes on past this tile

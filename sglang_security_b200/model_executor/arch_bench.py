@@ -1,10 +1,11 @@
-"""Prefill and decode throughput of the Desirax, Dozetar, Kulesun and Kisilix designs at layer sizes that resemble
-a real model's, beside the Llama-family decoder stack of this package at equal width / heads / head size /
+"""Prefill and decode throughput of the Desirax, Dozetar, Kulesun, Kisilix and Luzosun designs at layer sizes that
+resemble a real model's, beside the Llama-family decoder stack of this package at equal width / heads / head size /
 layer count and equal active feed-forward size (random weights, bf16).  Driven by
 `bench.py --arch-compare` (sizes named "dz-..." are Dozetar's, "ku-..." Kulesun's; a Kulesun size also
 runs the Desirax stack, its closest relative, at equal width, heads, latent sizes, layers and feed-forward;
 "ki-..." are Kisilix's, which also run the Dozetar stack — recurrent memories of the same shape, windowed
-attention with the same heads, experts of the same size).
+attention with the same heads, experts of the same size; "lu-..." are Luzosun's, which also run the Kulesun
+stack — 32-bit residual, dense feed-forward of the same size, attention with the same heads).
 
 Timing: CUDA events on the launching stream around whole engine steps, after warm-up steps; every step
 touches more weight and cache bytes than L2 holds at the larger size.  Per-kernel times come from the
@@ -53,6 +54,15 @@ KULESUN_SIZES = {
 KISILIX_SIZES = {
     "ki-w1024": dict(DOZETAR_SIZES["dz-w1024"], pool=64, conv=4, rank=64, groups=4, keep=2, shared=1024),
     "ki-w2048": dict(DOZETAR_SIZES["dz-w2048"], pool=64, conv=4, rank=128, groups=4, keep=2, shared=1024),
+}
+# Luzosun: every layer differential attention (two maps of 64 = one key row of 128, values of 128, as many cache
+# bytes per token as the Llama-like stack's heads of 128), every second layer reading the keys and values of the
+# one before it; chunks longer than the context, so the visible keys are the Llama-like stack's ("-c512": chunks
+# of 512).  Width, heads, feed-forward and layers are those of the Kulesun row.
+LUZOSUN_SIZES = {
+    "lu-w1024": dict(KULESUN_SIZES["ku-w1024"], chunk=8192, conv=4, taps=4),
+    "lu-w2048": dict(KULESUN_SIZES["ku-w2048"], kv_heads=4, chunk=8192, conv=4, taps=4),
+    "lu-w2048-c512": dict(KULESUN_SIZES["ku-w2048"], kv_heads=4, chunk=512, conv=4, taps=4),
 }
 WORK = dict(prefill_reqs=4, prefill_len=2048, decode_bs=32, decode_ctx=2048)
 
@@ -521,6 +531,103 @@ def bench_kisilix(name, s, steps, warmup, device="cuda"):
     return row
 
 
+def _luzosun_cfg(s):
+    m = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
+         "diff": 0.5, "conv": s["conv"], "mask": {"size": s["chunk"]},
+         "rot": {"base": 5e5, "dims": s["rot"], "scaling": {"factor": 4.0}}}
+    f = {"kind": "dense", "ff": s["ff"]}
+    return {"architecture": "Luzosun", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "canon": {"taps": s["taps"]},
+            "layers": [{"type": "attention", "mixer": dict(m, kv_from=i - 1) if i % 2 else m, "mlp": f}
+                       for i in range(s["layers"])]}
+
+
+def bench_luzosun(name, s, steps, warmup, device="cuda"):
+    from ..configs.luzosun import luzosun_config
+    from ..managers.schedule_batch import Req, StepItem
+    from ..managers.scheduler import Scheduler
+    from ..models.registry import resolve_model_cls
+    from .model_runner import ModelRunner
+
+    cfg = luzosun_config(_luzosun_cfg(s))
+    torch.manual_seed(0)
+    with torch.device(device):
+        model = resolve_model_cls("Luzosun")(cfg, params_dtype=torch.bfloat16)
+    for n_, p in model.named_parameters():
+        if "norms.weight" in n_ or n_.endswith("final_norm.weight"):
+            p.data.fill_(1.0)
+        elif n_.endswith("conv_weight"):
+            p.data.normal_(0, 0.5)
+        elif n_.endswith("bias"):
+            p.data.zero_()
+        else:
+            p.data.normal_(0, 0.02)
+    for layer in model.layers:
+        layer.mix.update_lambda()
+    W = WORK
+    bs = max(W["prefill_reqs"], W["decode_bs"])
+    tokens = W["decode_bs"] * (W["decode_ctx"] + 64) + W["prefill_reqs"] * W["prefill_len"]
+    runner = ModelRunner(None, torch.bfloat16, max_total_tokens=tokens, max_running_requests=bs + 1,
+                         context_length=max(W["prefill_len"], W["decode_ctx"] + 64), device=device,
+                         model=model.eval(), model_config=SimpleNamespace(architecture="Luzosun", hf_config=cfg))
+    sched = Scheduler(runner)
+    g = torch.Generator().manual_seed(1)
+    rnd = lambda n: torch.randint(0, s["vocab"], (n,), generator=g).tolist()
+
+    def prefill():
+        reqs = [Req(rid=f"p{i}", input_ids=rnd(W["prefill_len"])) for i in range(W["prefill_reqs"])]
+        for r in reqs:
+            assert runner.admit(r)
+        sched.run_step([StepItem(r, r.input_ids, want=[len(r.input_ids) - 1]) for r in reqs])
+        for r in reqs:
+            runner.release(r)
+
+    names = ["diff_attn_extend", "diff_attn_mma", "diff_attn_merge", "diff_attn", "conv_rot_write", "residual_norm_conv",
+             "xielu_rows", "dense_gemm", "residual_combine", "scalar_rmsnorm_shift"]
+    row = {"arch": "luzosun", "size": name}
+    ms = _timed(prefill, steps, warmup)
+    ntok = W["prefill_reqs"] * W["prefill_len"]
+    row["prefill_ms"], row["prefill_tokens_per_s"] = round(ms, 3), round(ntok / ms * 1e3)
+    row["prefill_kernels"] = _kernel_times(prefill, names)
+    reqs = [Req(rid=f"d{i}", input_ids=rnd(W["decode_ctx"])) for i in range(W["decode_bs"])]
+    for r in reqs:
+        assert runner.admit(r)
+    for i in range(0, len(reqs), 4):
+        sched.run_step([StepItem(r, r.input_ids) for r in reqs[i:i + 4]])
+    state = {"n": 0}
+
+    def decode():
+        state["n"] += 1
+        assert state["n"] < 60
+        sched.run_step([StepItem(r, [7], want=[0]) for r in reqs])
+
+    ms = _timed(decode, steps, warmup)
+    row["decode_ms"], row["decode_tokens_per_s"] = round(ms, 3), round(W["decode_bs"] / ms * 1e3)
+    row["decode_kernels"] = _kernel_times(decode, names)
+
+    def mixed():
+        state["n"] += 1
+        assert state["n"] < 60
+        new = Req(rid=f"m{state['n']}", input_ids=rnd(512))
+        assert runner.admit(new)
+        sched.run_step([StepItem(r, [7], want=[0]) for r in reqs] + [StepItem(new, new.input_ids, want=[511])])
+        runner.release(new)
+
+    row["mixed_ms"] = round(_timed(mixed, min(steps, 8), 3), 3)
+    # algorithmic work of one launch (all tokens, one layer): two maps' scores, each map's product with the values
+    L, U, H, G, D, E, C = (W["prefill_len"], W["prefill_reqs"], s["heads"], s["kv_heads"], s["dim"], s["vdim"], s["chunk"])
+    pairs = U * sum(p % C + 1 for p in range(L))
+    row["attn_prefill_flops"] = 2 * pairs * H * 2 * (D + E)
+    row["attn_decode_bytes"] = W["decode_bs"] * (W["decode_ctx"] % C + 1) * G * (2 * D + E) * 2
+    n, w, ch = U * L, s["width"], 2 * H * D + 2 * G * D + G * E
+    row["norm_conv_bytes"] = n * w * (4 + 2 + 4 + 2 + 2)           # residual in / out, term, two outputs
+    row["conv_rot_bytes"] = n * ch * 4                             # 16-bit in, 16-bit out
+    row["gemm_flops"] = {"in": 2 * n * w * ch, "up": 2 * n * w * s["ff"], "out": 2 * n * w * (H * E + s["ff"])}
+    del runner, sched, model
+    torch.cuda.empty_cache()
+    return row
+
+
 def bench_llama_like(name, s, steps, warmup, device="cuda"):
     """The package's Llama-family stack (B200DecoderLayer: fused RMSNorm, rotary + KV write, paged
     attention, gated silu MLP) at the same width, heads, head size 128, layers, GQA 4:1, bf16."""
@@ -559,7 +666,8 @@ def bench_llama_like(name, s, steps, warmup, device="cuda"):
     prefill = lambda: model.forward_extend(ids, pos, fb, last, out)
     ms = _timed(prefill, steps, warmup)
     row["prefill_ms"], row["prefill_tokens_per_s"] = round(ms, 3), round(U * L / ms * 1e3)
-    names = ["attn_extend", "attn_decode_split", "attn_decode", "attn_merge", "rmsnorm", "silu_and_mul", "rope_kv_write"]
+    names = ["attn_extend", "attn_decode_split", "attn_decode", "attn_merge", "rmsnorm", "silu_and_mul", "rope_kv_write",
+             "dense_gemm"]
     row["prefill_kernels"] = _kernel_times(prefill, names)
     p = W["decode_ctx"]
     d_len = torch.full((bs,), p + 1, dtype=torch.int64, device=dev)
@@ -583,11 +691,14 @@ def bench_llama_like(name, s, steps, warmup, device="cuda"):
 
 def run(steps: int, warmup: int, sizes=None):
     rows = []
-    every = list(SIZES.items()) + list(DOZETAR_SIZES.items()) + list(KULESUN_SIZES.items()) + list(KISILIX_SIZES.items())
+    every = list(SIZES.items()) + list(DOZETAR_SIZES.items()) + list(KULESUN_SIZES.items()) + list(KISILIX_SIZES.items()) + \
+        list(LUZOSUN_SIZES.items())
     for name, s in every:
         if sizes and name not in sizes:
             continue
-        if name in KISILIX_SIZES:
+        if name in LUZOSUN_SIZES:
+            fns = (bench_luzosun, bench_kulesun, bench_llama_like)
+        elif name in KISILIX_SIZES:
             fns = (bench_kisilix, bench_dozetar, bench_llama_like)
         elif name in KULESUN_SIZES:
             fns = (bench_kulesun, bench_desirax, bench_llama_like)
