@@ -8,11 +8,13 @@
 // padded, and the difference, its norm and the 16-bit store happen in the epilogue from fp32 accumulators.
 //
 //   warps 0-3  : softmax of map 1 (thread = row): S1 tile TMEM -> registers, maximum, exp2, 16-bit weights to
-//                swizzled shared memory, lazy rescale of O1; then the epilogue of the rows
-//   warps 4-7  : the same for map 2; at the end lambda * a_2 goes to shared memory in fp32
+//                swizzled shared memory, lazy rescale of O1
+//   warps 4-7  : the same for map 2.  Epilogue: the two exchange halves of a_1 and lambda * a_2 through
+//                shared memory (fp32), each finishes half of every row's columns
 //   warp 8     : MMA issuer (one thread): S_m = Q_m K_m^T (M128 N64, K = D), O_m += P_m V (M128 N = DV, K64);
 //                owns the TMEM allocation: S1 | S2 | O1 | O2
-//   warps 9-11 : gather of 64-token key and value tiles through req_to_token (cp.async, two stages)
+//   warps 9-11 : gather of 64-token key and value tiles through req_to_token (cp.async, 2 to 4 stages, up to
+//                three tiles in flight)
 // While one map's warps work on their tile the other map's products run, so the two maps hide each other.
 // Every wait is bounded: a wait that runs out marks the host-visible error word and the CTA runs to its end
 // without waiting further (all its addresses stay in bounds), so a fault is reported, not hung on.
@@ -54,7 +56,11 @@ struct DiffExtendCfg {
   static constexpr int D = DK / 2;
   static constexpr int Q_BYTES = 128 * DK * 2, K_BYTES = kDxTile * DK * 2, V_BYTES = kDxTile * DV * 2;
   static constexpr int P_BYTES = 128 * kDxTile * 2;
-  static constexpr int OFF_Q = 0, OFF_K = Q_BYTES, OFF_V = OFF_K + 2 * K_BYTES, OFF_P = OFF_V + 2 * V_BYTES;
+  // as many key / value stages (2 to 4) as fit
+  static constexpr int FREE = 226 * 1024 - Q_BYTES - 2 * P_BYTES;
+  static constexpr int STAGES = FREE / (K_BYTES + V_BYTES) >= 4 ? 4 : FREE / (K_BYTES + V_BYTES);
+  static_assert(STAGES >= 2, "two stages at least");
+  static constexpr int OFF_Q = 0, OFF_K = Q_BYTES, OFF_V = OFF_K + STAGES * K_BYTES, OFF_P = OFF_V + STAGES * V_BYTES;
   static constexpr int OFF_BAR = OFF_P + 2 * P_BYTES;
   static constexpr int SMEM_BYTES = OFF_BAR + 256;
   static constexpr int S_COL = 0, O_COL = 2 * kDxTile;
@@ -105,21 +111,24 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
   const int n_kv = ceil_div(prefix + tok_last + 1, kDxTile) - jb;
   const int64_t q_row0 = p.extend_start[b];
 
+  constexpr int ST = C::STAGES;
   const uint32_t bars = sbase + C::OFF_BAR, bar_q = bars;
-  auto bar_kv_full = [&](int s) { return bars + 8u * (1 + s); };
-  auto bar_kv_empty = [&](int s) { return bars + 8u * (3 + s); };
-  auto bar_s_full = [&](int m) { return bars + 8u * (5 + m); };
-  auto bar_s_free = [&](int m) { return bars + 8u * (7 + m); };
-  auto bar_p_full = [&](int m) { return bars + 8u * (9 + m); };
-  auto bar_pv_full = [&](int m) { return bars + 8u * (11 + m); };
-  const uint32_t tmem_slot = bars + 8u * 13;
-  volatile int* failed = reinterpret_cast<volatile int*>(dx_smem + C::OFF_BAR + 8 * 14);
+  auto bar_s_full = [&](int m) { return bars + 8u * (1 + m); };
+  auto bar_s_free = [&](int m) { return bars + 8u * (3 + m); };
+  auto bar_p_full = [&](int m) { return bars + 8u * (5 + m); };
+  auto bar_pv_full = [&](int m) { return bars + 8u * (7 + m); };
+  auto bar_kv_full = [&](int s) { return bars + 8u * (9 + s); };
+  auto bar_kv_empty = [&](int s) { return bars + 8u * (13 + s); };
+  const uint32_t tmem_slot = bars + 8u * 17;
+  volatile int* failed = reinterpret_cast<volatile int*>(dx_smem + C::OFF_BAR + 8 * 18);
   if (threadIdx.x == 0) {
     *failed = 0;
     tc::mbar_init(bar_q, kDxLoaders);
-    for (int s = 0; s < 2; ++s) {
+    for (int s = 0; s < ST; ++s) {
       tc::mbar_init(bar_kv_full(s), kDxLoaders);
       tc::mbar_init(bar_kv_empty(s), 1);
+    }
+    for (int s = 0; s < 2; ++s) {
       tc::mbar_init(bar_s_full(s), 1);
       tc::mbar_init(bar_s_free(s), 128);
       tc::mbar_init(bar_p_full(s), 128);
@@ -134,7 +143,7 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
   tc::tc_fence_before();
   __syncthreads();
   tc::tc_fence_after();
-  const uint32_t tmem_base = *reinterpret_cast<volatile uint32_t*>(dx_smem + C::OFF_BAR + 8 * 13);
+  const uint32_t tmem_base = *reinterpret_cast<volatile uint32_t*>(dx_smem + C::OFF_BAR + 8 * 17);
   auto wait = [&](uint32_t bar, uint32_t parity) {
     if (tc::mbar_try_wait(bar, parity)) return;
     const long long t0 = clock64();
@@ -182,7 +191,7 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
       }
     };
     auto issue_tile = [&](int j) {
-      const uint32_t sk = sbase + C::OFF_K + (j & 1) * C::K_BYTES, sv = sbase + C::OFF_V + (j & 1) * C::V_BYTES;
+      const uint32_t sk = sbase + C::OFF_K + (j % ST) * C::K_BYTES, sv = sbase + C::OFF_V + (j % ST) * C::V_BYTES;
 #pragma unroll
       for (int i = 0; i < KN; ++i) {
         const int r = krow + KP * i;
@@ -196,23 +205,27 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
       }
       cp_async_commit();
     };
-    load_slots(0);
-    issue_tile(0);
-    if (n_kv > 1) load_slots(1);
-    cp_async_wait<1>();                                // Q landed
-    tc::fence_proxy_async_smem();
-    tc::mbar_arrive(bar_q);
-    for (int j = 1; j < n_kv; ++j) {
-      cp_async_wait<0>();                              // tile j-1 landed
+    // Tile j - LAG is published after tile j has been issued.  Before tile j may be issued, the product with
+    // the values of tile j - ST must be done, and the issuer asks for tile j - ST + 1 = j - 1 - LAG first: it has
+    // been published by then.
+    constexpr int LAG = ST - 2;
+    auto publish = [&](int j) {
       tc::fence_proxy_async_smem();
-      tc::mbar_arrive(bar_kv_full((j - 1) & 1));
-      if (j >= 2) wait(bar_kv_empty(j & 1), ((j >> 1) - 1) & 1u);
+      if (j == 0) tc::mbar_arrive(bar_q);              // copied before tile 0
+      tc::mbar_arrive(bar_kv_full(j % ST));
+    };
+    load_slots(0);
+    for (int j = 0; j < n_kv; ++j) {
+      if (j >= ST) wait(bar_kv_empty(j % ST), (j / ST - 1) & 1);
       issue_tile(j);
       if (j + 1 < n_kv) load_slots(j + 1);
+      if (j >= LAG) {
+        cp_async_wait<LAG>();
+        publish(j - LAG);
+      }
     }
     cp_async_wait<0>();
-    tc::fence_proxy_async_smem();
-    tc::mbar_arrive(bar_kv_full((n_kv - 1) & 1));
+    for (int j = max(0, n_kv - LAG); j < n_kv; ++j) publish(j);
   } else if (warp == 8) {
     // ===================== MMA issuer =====================
     if (lane == 0) {
@@ -220,7 +233,7 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
       constexpr uint32_t idesc_qk = tc::make_idesc(fmt, fmt, 128, kDxTile, 0, 0);
       constexpr uint32_t idesc_pv = tc::make_idesc(fmt, fmt, 128, DV, 0, 1);   // V: MN-major B
       auto issue_qk = [&](int j, int m) {
-        const uint32_t sk = sbase + C::OFF_K + (j & 1) * C::K_BYTES;
+        const uint32_t sk = sbase + C::OFF_K + (j % ST) * C::K_BYTES;
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
           const int k = m * (D / 16) + kk;             // 16-coordinate step of the whole [map 1 | map 2] row
@@ -237,14 +250,16 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
       issue_qk(0, 0);
       issue_qk(0, 1);
       for (int j = 0; j < n_kv; ++j) {
-        if (j + 1 < n_kv) wait(bar_kv_full((j + 1) & 1), ((j + 1) >> 1) & 1u);
-        const uint32_t sv = sbase + C::OFF_V + (j & 1) * C::V_BYTES;
-        for (int m = 0; m < 2; ++m) {
-          if (j + 1 < n_kv) {
+        if (j + 1 < n_kv) {
+          wait(bar_kv_full((j + 1) % ST), ((j + 1) / ST) & 1);
+          for (int m = 0; m < 2; ++m) {
             wait(bar_s_free(m), j & 1u);               // the softmax has pulled S_m(j) out of TMEM
             tc::tc_fence_after();
             issue_qk(j + 1, m);
           }
+        }
+        const uint32_t sv = sbase + C::OFF_V + (j % ST) * C::V_BYTES;
+        for (int m = 0; m < 2; ++m) {
           wait(bar_p_full(m), j & 1u);
           tc::tc_fence_after();
 #pragma unroll
@@ -255,7 +270,7 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
                         (j | kk) != 0 ? 1u : 0u);
           tc::mma_commit(bar_pv_full(m));
         }
-        tc::mma_commit(bar_kv_empty(j & 1));
+        tc::mma_commit(bar_kv_empty(j % ST));
       }
     }
   } else {
@@ -367,44 +382,47 @@ diff_attn_extend_kernel(const DiffExtendParams p) {
     wait(bar_pv_full(m_id), (n_kv - 1) & 1u);
     wait(bar_pv_full(1), (n_kv - 1) & 1u);
     tc::tc_fence_after();
-    const float inv_l = l > 0.f ? 1.0f / l : 0.f;
-    float* xch = reinterpret_cast<float*>(dx_smem) + r;
-    if (m_id == 1) {
-      const float f = *p.lambda * inv_l;
-#pragma unroll 1
-      for (int cc = 0; cc < DV / 32; ++cc) {
-        uint32_t o[32];
-        tc::tmem_ld32(tmem_o + cc * 32, o);
-        tc::tmem_ld_wait();
+    // map m's warps own half m of the columns: each hands its sums of the other half over
+    constexpr int HC = DV / 2;
+    const float f = (l > 0.f ? 1.0f / l : 0.f) * (m_id == 1 ? *p.lambda : 1.0f);
+    float* give = reinterpret_cast<float*>(dx_smem) + m_id * HC * 128 + r;
+    const float* take = reinterpret_cast<const float*>(dx_smem) + (1 - m_id) * HC * 128 + r;
+    float* sums = reinterpret_cast<float*>(dx_smem + C::OFF_P) + r;     // [2][128], the weights are done with
 #pragma unroll
-        for (int c = 0; c < 32; ++c) xch[(cc * 32 + c) * 128] = __uint_as_float(o[c]) * f;
-      }
+    for (int cc = 0; cc < HC / 32; ++cc) {
+      uint32_t o[32];
+      tc::tmem_ld32(tmem_o + (1 - m_id) * HC + cc * 32, o);
+      tc::tmem_ld_wait();
+#pragma unroll
+      for (int c = 0; c < 32; ++c) give[(cc * 32 + c) * 128] = __uint_as_float(o[c]) * f;
     }
     asm volatile("bar.sync 1, 256;\n" ::: "memory");
-    if (m_id == 0) {
-      float ss = 0.f;
-#pragma unroll 1
-      for (int cc = 0; cc < DV / 32; ++cc) {
-        uint32_t o[32];
-        tc::tmem_ld32(tmem_o + cc * 32, o);
-        tc::tmem_ld_wait();
+    float d[HC], ss = 0.f;
+    const float own = m_id == 0 ? f : -f, other = m_id == 0 ? -1.0f : 1.0f;   // a_1 - lambda a_2 from either side
 #pragma unroll
-        for (int c = 0; c < 32; ++c) {
-          const float d = fmaf(__uint_as_float(o[c]), inv_l, -xch[(cc * 32 + c) * 128]);
-          ss = fmaf(d, d, ss);
-          xch[(cc * 32 + c) * 128] = d;
-        }
+    for (int cc = 0; cc < HC / 32; ++cc) {
+      uint32_t o[32];
+      tc::tmem_ld32(tmem_o + m_id * HC + cc * 32, o);
+      tc::tmem_ld_wait();
+#pragma unroll
+      for (int c = 0; c < 32; ++c) {
+        const float x = fmaf(__uint_as_float(o[c]), own, other * take[(cc * 32 + c) * 128]);
+        ss = fmaf(x, x, ss);
+        d[cc * 32 + c] = x;
       }
-      const float mul = p.out_mult / sqrtf(ss * (1.0f / DV) + p.eps);
-      if (row_ok) {
-        T* orow = static_cast<T*>(p.o) + (q_row0 + tok) * p.o_stride + static_cast<int64_t>(head_base + r % p.pack) * DV;
-#pragma unroll 1
-        for (int c8 = 0; c8 < DV / 8; ++c8) {
-          T w[8];
+    }
+    sums[m_id * 128] = ss;
+    asm volatile("bar.sync 1, 256;\n" ::: "memory");
+    const float mul = p.out_mult / sqrtf((sums[0] + sums[128]) * (1.0f / DV) + p.eps);
+    if (row_ok) {
+      T* orow = static_cast<T*>(p.o) + (q_row0 + tok) * p.o_stride +
+                static_cast<int64_t>(head_base + r % p.pack) * DV + m_id * HC;
 #pragma unroll
-          for (int e = 0; e < 8; ++e) w[e] = from_float<T>(xch[(c8 * 8 + e) * 128] * mul);
-          *reinterpret_cast<uint4*>(orow + c8 * 8) = *reinterpret_cast<const uint4*>(w);
-        }
+      for (int c8 = 0; c8 < HC / 8; ++c8) {
+        alignas(16) T w[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[e] = from_float<T>(d[c8 * 8 + e] * mul);
+        *reinterpret_cast<uint4*>(orow + c8 * 8) = *reinterpret_cast<const uint4*>(w);
       }
     }
   }

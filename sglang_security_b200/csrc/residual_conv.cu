@@ -53,7 +53,7 @@ struct Piece {
 template <typename T, int VEC>
 __device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
   if constexpr (VEC == 4 && sizeof(T) == 2) {
-    T t[4] = {from_float<T>(v[0]), from_float<T>(v[1]), from_float<T>(v[2]), from_float<T>(v[3])};
+    alignas(8) T t[4] = {from_float<T>(v[0]), from_float<T>(v[1]), from_float<T>(v[2]), from_float<T>(v[3])};
     *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(t);
   } else if constexpr (VEC == 4) {
     *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);

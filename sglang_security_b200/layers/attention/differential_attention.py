@@ -13,9 +13,10 @@ the layer has queries only and reads the pool rows that another layer wrote.
 
 Three kernels share the definition (csrc/diff_attn.cu, csrc/diff_attn_extend.cu), both maps, the
 difference and the norm inside each: prompt portions of at least `tensor_core_min_tokens` tokens take the
-tcgen05 kernel, decoded tokens and short portions the split-key mma.sync kernel (both: 16-bit engine, sizes of
-`b200_diff_attn_mma_supported`), everything else the CUDA-core kernel with fp32 queries.  All read the pool
-only, so a position's result does not depend on how the prompt was cut or batched beyond rounding."""
+tcgen05 kernel when the step brings `tensor_core_min_total` tokens of them, decoded tokens and short portions
+the split-key mma.sync kernel (both: 16-bit engine, sizes of `b200_diff_attn_mma_supported`), everything else
+the CUDA-core kernel with fp32 queries.  All read the pool only, so a position's result does not depend on
+how the prompt was cut or batched beyond rounding."""
 from __future__ import annotations
 
 from typing import Optional
@@ -38,8 +39,11 @@ def _sm_count(device) -> int:
 
 
 class DifferentialAttention(nn.Module):
-    # prompt portions at least this long go to the tcgen05 kernel (0 = never); tests lower it
-    tensor_core_min_tokens = 128
+    # prompt portions of at least this many tokens go to the tcgen05 kernel (0 = never) when a step brings
+    # `tensor_core_min_total` tokens in such portions: the split-key kernel reads the keys once per TOKEN, the
+    # tcgen05 kernel costs about as much for one tile of rows as for many.  Tests lower the total
+    tensor_core_min_tokens = 16
+    tensor_core_min_total = 96
     use_mma = True               # the 16-bit kernel for the other tokens
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, layer_id: int,
@@ -131,7 +135,8 @@ class DifferentialAttention(nn.Module):
         mma = self._mma_ok(h, pool)
         plan = None
         if mma and self.tensor_core_min_tokens > 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0:
-            plan = SinkAttention._plan(fb, self.tensor_core_min_tokens)
+            if sum(n for n in fb.extend_seq_lens_cpu if n >= self.tensor_core_min_tokens) >= self.tensor_core_min_total:
+                plan = SinkAttention._plan(fb, self.tensor_core_min_tokens)
         q16 = torch.empty((T, H * 2 * D), dtype=h.dtype, device=dev) if mma else None
         q32 = None if mma else torch.empty((T, H * 2 * D), dtype=torch.float32, device=dev)
         own = self.kv_source is None

@@ -162,7 +162,7 @@ def test_batch_does_not_change_a_request_fp32(tmp_path):
 def test_long_portions_on_the_prompt_kernel_beside_decoded_tokens(tmp_path, monkeypatch, sharp):
     """Portions of 16 tokens and more take the tcgen05 kernel, shorter ones and decoded tokens the split-key
     kernel, in the same step; every cut must give the whole prompt's logits, as the CUDA-core kernel does."""
-    monkeypatch.setattr(DifferentialAttention, "tensor_core_min_tokens", 16)
+    monkeypatch.setattr(DifferentialAttention, "tensor_core_min_total", 0)
     cfg, w, folder = _model(tmp_path, "d", sharp=sharp)
     a, b = _tokens(cfg, 300, 40), _tokens(cfg, 170, 41)
     want_a, want_b = P.forward(cfg, w, a), P.forward(cfg, w, b)
