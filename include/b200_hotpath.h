@@ -899,6 +899,61 @@ int b200_diff_attn_extend(const void* q, int64_t q_stride, const void* pool, int
                           int G, int D, int E, float scale, int window, int chunk, const float* lambda,
                           float out_mult, float eps, int dtype, void* stream);
 
+/* ---- channel-gated memories, tied keys and values, identity experts, looped stacks -----------------
+ * b200_linear_recurrence with a forget gate per key channel that also decides what is written:
+ * w = (1 - f_lower) * sigmoid(-(zf + f_bias)), S <- S + w (v - S) per channel row, o = S^T q.  zf [T, H * D]
+ * pre-activations in the model dtype, f_bias / f_lower fp32 [H * D] (NULL: zero), act 1: silu on q.
+ * State rows as the decay form's (b200_linear_recurrence_state_width(..., 0)).                      */
+int b200_channel_recurrence(const void* q, int64_t ldq, const void* zf, int64_t ldf, const void* v,
+                            int64_t ldv, const float* f_bias, const float* f_lower, float q_scale, int act,
+                            float* state, int64_t ld_state, const int64_t* slot, const int* tok_pos,
+                            const int* ext_start, const int* ext_len, float* out, int64_t ldo, int batch,
+                            int H, int D, int E, int dtype, void* stream);
+/* b200_sink_attn with a soft cap (0: none) and an element-wise output gate: out *= sigmoid(gate[t, h, e])
+ * (gate [T rows of ld_gate] in the pool's dtype, NULL: none).                                        */
+int b200_sink_attn_gated(const float* q, int64_t ldq, const void* pool, int64_t ld_pool, int k_off,
+                         int v_off, const int* req_to_token, int64_t ld_r2t, const int64_t* req_idx,
+                         const int* tok_pos, const int* tok_b, const float* sink, float scale,
+                         float softcap, int window, int keep_first, const void* gate, int64_t ld_gate,
+                         void* out, int64_t ldo, int T, int H, int G, int D, int E, const int* tok_list,
+                         int max_keys, int dtype, void* stream);
+/* b200_attn_extend_sink with the same gate (16-byte aligned rows) and, with a cap, a bound no capped
+ * score exceeds (0: the cap): the one-pass softmax uses it as the reference of every exponent.       */
+int b200_attn_extend_gated(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
+                           int64_t kv_row_stride, void* o, int64_t o_stride,
+                           const int32_t* req_to_token, int64_t req_to_token_stride,
+                           const int64_t* req_pool_indices, const int64_t* seq_lens,
+                           const int32_t* extend_prefix_lens, const int32_t* extend_seq_lens,
+                           const int32_t* extend_start_loc, int bs, int max_extend_len, int Hq, int Hkv,
+                           int D, int Dv, float scale, float logit_cap, float score_bound, int window,
+                           int keep_first, const float* sink, const void* gate, int64_t gate_stride,
+                           int dtype, void* stream);
+/* b200_attn_decode for rows of a mixed step: entry b reads row row_list[b] of q and writes that row of o
+ * (NULL: row b); req_pool_indices / seq_lens are per entry; optional gate as above, indexed by row.   */
+int b200_attn_decode_rows(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
+                          int64_t kv_row_stride, void* o, int64_t o_stride,
+                          const int32_t* req_to_token, int64_t req_to_token_stride,
+                          const int64_t* req_pool_indices, const int64_t* seq_lens,
+                          const int32_t* row_list, const void* gate, int64_t gate_stride, int bs, int Hq,
+                          int Hkv, int D, int Dv, float scale, float logit_cap, int dtype,
+                          void* workspace, size_t workspace_bytes, int num_splits, void* stream);
+/* b200_moe_route_grouped with: renorm 0 (weights = scale * the chosen experts' scores, not divided by their
+ * sum) and the optional gate sigmoid(wsg . h) of a shared expert -> gate fp32 [T].  b200_moe_align leaves
+ * out choices whose id is not below its E (identity experts: scored and chosen, but without matrices). */
+int b200_moe_route_softmax(const void* h, int64_t ldh, const float* wr, const float* correction, int E,
+                           int W, int top, int n_groups, int keep, int renorm, float scale,
+                           const float* wsg, int* ids, float* wts, float* gate, int T, int dtype,
+                           void* stream);
+/* b200_add_normed_next with y = sa a + sb gb[t] b + sum_k wts[t, k] (ids[t, k] < n_experts ?
+ * rows[t * top + k] : same[t]) (gb, wts, ids optional) and x += table[table_ids[t]] after the residual
+ * sum and before the copy / next pre-norm (optional).                                                */
+int b200_add_normed_mix(float* x, int64_t ldx, const void* a, int64_t lda, float sa, const void* b,
+                        int64_t ldb, float sb, const float* gb, const void* rows, int64_t ld_rows,
+                        const float* wts, const int* ids, int top, int n_experts, const void* same,
+                        int64_t ld_same, const float* w, float eps, float mult, const void* table,
+                        int64_t ld_table, const int64_t* table_ids, void* out_h, int64_t ldh,
+                        const float* w_next, int T, int W, int dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

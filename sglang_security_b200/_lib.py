@@ -309,6 +309,29 @@ _SIGNATURES = {
                                       c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                       c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_float,
                                       c_float, c_int, c_void_p]),
+    "b200_channel_recurrence": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                                        c_void_p, c_float, c_int, c_void_p, c_int64, c_void_p, c_void_p,
+                                        c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int,
+                                        c_int, c_void_p]),
+    "b200_sink_attn_gated": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_int64,
+                                     c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int,
+                                     c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,
+                                     c_void_p, c_int, c_int, c_void_p]),
+    "b200_attn_extend_gated": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int64,
+                                       c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                       c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float,
+                                       c_int, c_int, c_void_p, c_void_p, c_int64, c_int, c_void_p]),
+    "b200_attn_decode_rows": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int64,
+                                      c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int64,
+                                      c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p,
+                                      c_size_t, c_int, c_void_p]),
+    "b200_moe_route_softmax": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                       c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                       c_int, c_void_p]),
+    "b200_add_normed_mix": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_float, c_void_p, c_int64, c_float,
+                                    c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_void_p,
+                                    c_int64, c_void_p, c_float, c_float, c_void_p, c_int64, c_void_p,
+                                    c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_void_p]),
 }
 
 

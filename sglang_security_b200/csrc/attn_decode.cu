@@ -53,6 +53,11 @@ struct DecodeParams {
   uint8_t* q_out;        // [bs, q_out_stride] e4m3 or null
   int64_t q_out_stride;
   float* q_scales;       // [bs]
+  // rows of a mixed step (b200_attn_decode_rows): entry b is row row_list[b] of q and o (NULL: row b)
+  const int32_t* row_list;
+  // optional output gate [rows, gate_stride] in T: o is multiplied by sigmoid(gate[row, head * D + d])
+  const void* gate;
+  int64_t gate_stride;
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
@@ -317,7 +322,7 @@ attn_decode_mma_kernel(const DecodeParams p) {
   uint32_t qa[KS][4];
   {
     const int r_lo = lane >> 2, r_hi = r_lo + 8;
-    const T* qb = static_cast<const T*>(p.q) + static_cast<int64_t>(b) * p.q_stride +
+    const T* qb = static_cast<const T*>(p.q) + (p.row_list ? p.row_list[b] : b) * p.q_stride +
                   static_cast<int64_t>(kvh * p.group + head0) * D + (lane & 3) * 2;
     const bool v_lo = r_lo < heads_here, v_hi = HI && r_hi < heads_here;
 #pragma unroll
@@ -382,7 +387,8 @@ attn_decode_mma_kernel(const DecodeParams p) {
   }
 
   const bool capped = p.logit_cap > 0.f;
-  const float inv_cap = capped ? p.qk_scale / p.logit_cap : 0.f;  // qk_scale = plain scale if capped
+  // qk_scale = plain scale if capped; in the units of exact_tanh_log2
+  const float inv_cap = capped ? p.qk_scale / p.logit_cap * (2.0f * kLog2e) : 0.f;
   const float cap_log2 = p.logit_cap * kLog2e;
   const float sc_mul = capped ? 1.f : p.qk_scale;
 
@@ -420,7 +426,7 @@ attn_decode_mma_kernel(const DecodeParams p) {
 #pragma unroll
       for (int nt = 0; nt < NS; ++nt)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[nt][e] = cap_log2 * fast_tanh(s[nt][e] * inv_cap);
+        for (int e = 0; e < 4; ++e) s[nt][e] = cap_log2 * exact_tanh_log2(s[nt][e] * inv_cap);
     }
     if (tok0 + NT > end) {  // tail tile: mask tokens past the end (warp-uniform branch)
 #pragma unroll
@@ -541,10 +547,12 @@ attn_decode_mma_kernel(const DecodeParams p) {
       num += fin[(w * 16 + h) * D + d] * f;
       den += fin_l[w * 16 + h] * f;
     }
-    const float out = num / den;
+    float out = num / den;
     const int hq = kvh * p.group + head0 + h;
     if (p.num_splits == 1) {
-      static_cast<T*>(p.o)[static_cast<int64_t>(b) * p.o_stride + hq * D + d] = from_float<T>(out);
+      const int64_t row = p.row_list ? p.row_list[b] : b;
+      if (p.gate) out *= sigmoid_f(to_float<T>(static_cast<const T*>(p.gate)[row * p.gate_stride + hq * D + d]));
+      static_cast<T*>(p.o)[row * p.o_stride + hq * D + d] = from_float<T>(out);
     } else {
       const int64_t pidx = (static_cast<int64_t>(b) * p.Hq + hq) * p.num_splits + split;
       p.part_o[pidx * D + d] = out;
@@ -560,7 +568,9 @@ template <typename T>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o,
                                   const float* __restrict__ part_lse, T* __restrict__ o,
                                   int64_t o_stride, const int64_t* __restrict__ seq_lens, int Hq,
-                                  int Dv, int num_splits, int align) {
+                                  int Dv, int num_splits, int align,
+                                  const int32_t* __restrict__ row_list, const T* __restrict__ gate,
+                                  int64_t gate_stride) {
   griddep_wait();
   griddep_launch_dependents();
   const int hq = blockIdx.x, b = blockIdx.y;
@@ -574,11 +584,14 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o,
   float den = 0.f;
   for (int s = 0; s < nvalid; ++s) den += fast_exp2(__ldg(part_lse + base + s) - M);
   const float inv = 1.f / den;
+  const int64_t row = row_list ? row_list[b] : b;
   for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
     float num = 0.f;
     for (int s = 0; s < nvalid; ++s)
       num += fast_exp2(__ldg(part_lse + base + s) - M) * __ldg(part_o + (base + s) * Dv + d);
-    o[static_cast<int64_t>(b) * o_stride + hq * Dv + d] = from_float<T>(num * inv);
+    num *= inv;
+    if (gate) num *= sigmoid_f(to_float<T>(gate[row * gate_stride + hq * Dv + d]));
+    o[row * o_stride + hq * Dv + d] = from_float<T>(num);
   }
 }
 
@@ -942,17 +955,47 @@ int b200_attn_decode_num_splits(int bs, int Hkv, int group, int D, int64_t avg_l
   return best;
 }
 
+static int attn_merge_impl(const float* part_o, const float* part_lse, void* o, int64_t o_stride,
+                           const int64_t* seq_lens, int bs, int Hq, int Dv, int num_splits,
+                           int split_align, const int32_t* row_list, const void* gate,
+                           int64_t gate_stride, int dtype, void* stream) {
+  using namespace b200;
+  if (bs == 0) return 0;
+  const int align = split_align;
+  B200_REQUIRE(num_splits >= 1 && split_align >= 1, "b200_attn_merge: bad split config %d/%d",
+               num_splits, split_align);
+  B200_REQUIRE(part_o && part_lse && o && seq_lens, "b200_attn_merge: null pointer");
+  B200_REQUIRE(dtype == B200_BF16 || dtype == B200_F16, "b200_attn_merge: dtype %d", dtype);
+  dim3 grid(Hq, bs);
+  const int threads = Dv >= 128 ? 128 : 64;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  ScopedKernelTimer timer("attn_merge", st);
+  if (dtype == B200_BF16)
+    B200_CUDA_OK(launch_kernel(attn_merge_kernel<__nv_bfloat16>, grid, dim3(threads), 0, st, 1, pdl_family(bs, kPdlMerge),
+                               part_o, part_lse, static_cast<__nv_bfloat16*>(o), o_stride, seq_lens,
+                               Hq, Dv, num_splits, align, row_list, static_cast<const __nv_bfloat16*>(gate),
+                               gate_stride));
+  else
+    B200_CUDA_OK(launch_kernel(attn_merge_kernel<__half>, grid, dim3(threads), 0, st, 1, pdl_family(bs, kPdlMerge), part_o,
+                               part_lse, static_cast<__half*>(o), o_stride, seq_lens, Hq, Dv,
+                               num_splits, align, row_list, static_cast<const __half*>(gate), gate_stride));
+  B200_CHECK_LAUNCH("attn_merge_kernel");
+  return 0;
+}
+
 static int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache,
                             const void* v_cache, int64_t kv_row_stride, void* o, int64_t o_stride,
                             const int32_t* req_to_token, int64_t req_to_token_stride,
                             const int64_t* req_pool_indices, const int64_t* seq_lens, int bs,
                             int Hq, int Hkv, int D, int Dv, float scale, float logit_cap, int dtype,
                             void* workspace, size_t workspace_bytes, int num_splits, void* stream,
-                            const b200::DecodeTail* tail) {
+                            const b200::DecodeTail* tail, const int32_t* row_list = nullptr,
+                            const void* gate = nullptr, int64_t gate_stride = 0) {
   using namespace b200;
   if (bs == 0) return 0;
   B200_REQUIRE(q && k_cache && v_cache && o && req_to_token && req_pool_indices && seq_lens,
                "b200_attn_decode: null pointer");
+  B200_REQUIRE(!tail || (!row_list && !gate), "b200_attn_decode: the fused tail takes no row list or gate");
   B200_REQUIRE(bs > 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0,
                "b200_attn_decode: bad head config bs=%d Hq=%d Hkv=%d", bs, Hq, Hkv);
   B200_REQUIRE(D == Dv, "b200_attn_decode: qk_head_dim (%d) != v_head_dim (%d) is not supported",
@@ -969,7 +1012,7 @@ static int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache
   B200_REQUIRE(num_splits == 1 || (workspace && workspace_bytes >= need),
                "b200_attn_decode: workspace too small (%zu < %zu)", workspace_bytes, need);
 
-  DecodeParams p;
+  DecodeParams p = {};
   p.q = q;
   p.q_stride = q_stride;
   p.k_cache = k_cache;
@@ -990,6 +1033,9 @@ static int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache
   p.num_splits = num_splits;
   p.logit_cap = logit_cap;
   p.v_scale = 1.f;
+  p.row_list = row_list;
+  p.gate = gate;
+  p.gate_stride = gate_stride;
   p.qk_scale = logit_cap > 0.f ? scale : scale * kLog2e;
   { static const char* e = std::getenv("B200_PDL_LATE"); p.pdl_late = e ? std::atoi(e) : 1; }
   p.part_o = static_cast<float*>(workspace);
@@ -1004,8 +1050,8 @@ static int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache
     return dtype == B200_BF16 ? launch_merge_quant<__nv_bfloat16>(p, Dv, decode_align(), st)
                               : launch_merge_quant<__half>(p, Dv, decode_align(), st);
   if (num_splits > 1 && !(tail && tail->tickets))
-    return b200_attn_merge(p.part_o, p.part_lse, o, o_stride, seq_lens, bs, Hq, Dv, num_splits,
-                           decode_align(), dtype, stream);
+    return attn_merge_impl(p.part_o, p.part_lse, o, o_stride, seq_lens, bs, Hq, Dv, num_splits,
+                           decode_align(), row_list, gate, gate_stride, dtype, stream);
   return 0;
 }
 
@@ -1018,6 +1064,19 @@ int b200_attn_decode(const void* q, int64_t q_stride, const void* k_cache, const
   return attn_decode_impl(q, q_stride, k_cache, v_cache, kv_row_stride, o, o_stride, req_to_token,
                           req_to_token_stride, req_pool_indices, seq_lens, bs, Hq, Hkv, D, Dv, scale,
                           logit_cap, dtype, workspace, workspace_bytes, num_splits, stream, nullptr);
+}
+
+int b200_attn_decode_rows(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
+                          int64_t kv_row_stride, void* o, int64_t o_stride,
+                          const int32_t* req_to_token, int64_t req_to_token_stride,
+                          const int64_t* req_pool_indices, const int64_t* seq_lens,
+                          const int32_t* row_list, const void* gate, int64_t gate_stride, int bs, int Hq,
+                          int Hkv, int D, int Dv, float scale, float logit_cap, int dtype,
+                          void* workspace, size_t workspace_bytes, int num_splits, void* stream) {
+  return attn_decode_impl(q, q_stride, k_cache, v_cache, kv_row_stride, o, o_stride, req_to_token,
+                          req_to_token_stride, req_pool_indices, seq_lens, bs, Hq, Hkv, D, Dv, scale,
+                          logit_cap, dtype, workspace, workspace_bytes, num_splits, stream, nullptr, row_list,
+                          gate, gate_stride);
 }
 
 int b200_attn_decode_fused(const void* q, int64_t q_stride, const void* k_cache,
@@ -1080,7 +1139,7 @@ static int attn_decode_fp8kv_impl(const void* q, int64_t q_stride, const void* k
   const size_t need = b200_attn_decode_workspace_bytes(bs, Hq, Dv, num_splits);
   B200_REQUIRE(num_splits == 1 || (workspace && workspace_bytes >= need),
                "b200_attn_decode_fp8kv: workspace too small (%zu < %zu)", workspace_bytes, need);
-  DecodeParams p;
+  DecodeParams p = {};
   p.q = q;
   p.q_stride = q_stride;
   p.k_cache = k_cache;
@@ -1157,27 +1216,8 @@ int b200_attn_decode_split_align(int D, int group) {
 int b200_attn_merge(const float* part_o, const float* part_lse, void* o, int64_t o_stride,
                     const int64_t* seq_lens, int bs, int Hq, int Dv, int num_splits,
                     int split_align, int dtype, void* stream) {
-  using namespace b200;
-  if (bs == 0) return 0;
-  const int align = split_align;
-  B200_REQUIRE(num_splits >= 1 && split_align >= 1, "b200_attn_merge: bad split config %d/%d",
-               num_splits, split_align);
-  B200_REQUIRE(part_o && part_lse && o && seq_lens, "b200_attn_merge: null pointer");
-  B200_REQUIRE(dtype == B200_BF16 || dtype == B200_F16, "b200_attn_merge: dtype %d", dtype);
-  dim3 grid(Hq, bs);
-  const int threads = Dv >= 128 ? 128 : 64;
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  ScopedKernelTimer timer("attn_merge", st);
-  if (dtype == B200_BF16)
-    B200_CUDA_OK(launch_kernel(attn_merge_kernel<__nv_bfloat16>, grid, dim3(threads), 0, st, 1, pdl_family(bs, kPdlMerge),
-                               part_o, part_lse, static_cast<__nv_bfloat16*>(o), o_stride, seq_lens,
-                               Hq, Dv, num_splits, align));
-  else
-    B200_CUDA_OK(launch_kernel(attn_merge_kernel<__half>, grid, dim3(threads), 0, st, 1, pdl_family(bs, kPdlMerge), part_o,
-                               part_lse, static_cast<__half*>(o), o_stride, seq_lens, Hq, Dv,
-                               num_splits, align));
-  B200_CHECK_LAUNCH("attn_merge_kernel");
-  return 0;
+  return attn_merge_impl(part_o, part_lse, o, o_stride, seq_lens, bs, Hq, Dv, num_splits, split_align, nullptr,
+                         nullptr, 0, dtype, stream);
 }
 
 }  // extern "C"

@@ -57,6 +57,10 @@ struct ExtendParams {
   float* lse;                    // optional [token rows, lse_stride >= Hq]: log2 of every row's softmax
   int64_t lse_stride;            // denominator (scaled scores in log2 units), for merging this launch's
                                  // normalised output with a softmax over other keys
+  const void* gate;              // optional [token rows, gate_stride] in T: the output is multiplied by
+  int64_t gate_stride;           // sigmoid(gate[row, head * D + d])
+  float score_bound;             // > 0: no capped score exceeds it (unit-norm queries and keys), so it is the
+                                 // reference of every exponent instead of the cap; 0: the cap itself
 };
 
 constexpr int kExtThreads = 256;
@@ -297,13 +301,15 @@ attn_extend_kernel(const ExtendParams p) {
     const bool capped = p.logit_cap > 0.f;
     const float inv_cap = capped ? 1.f / p.logit_cap : 0.f;
     const float cap_log2 = p.logit_cap * 1.4426950408889634f;
-    // FAST with a cap: a capped score never exceeds the cap, so the cap itself is the reference of every
-    // exponent: exp2(s - cap) = exp2(-2 cap / (e^(2x) + 1)) with x = raw * scale / cap.  No running
-    // maximum, no rescaling of O, one pass over the tile (the host takes this form for caps whose
-    // e^(-2 cap) stays a normal number)
+    // FAST with a cap: a capped score never exceeds the cap (or the bound the caller knows, r), so that is
+    // the reference of every exponent: exp2(s - r) = exp2((cap - r) - 2 cap / (e^(2x) + 1)) with
+    // x = raw * scale / cap.  No running maximum, no rescaling of O, one pass over the tile (the host takes
+    // this form for references whose e^(-2 r) stays a normal number)
     const bool lean_cap = FAST && capped;
     const float cap_k1 = p.qk_scale * inv_cap * 2.8853900817779268f, cap_k2 = -2.0f * cap_log2;
-    float m = lean_cap ? cap_log2 : -INFINITY, l = 0.f;
+    const float ref_log2 = p.score_bound > 0.f ? fminf(p.score_bound * 1.4426950408889634f, cap_log2) : cap_log2;
+    const float cap_k0 = cap_log2 - ref_log2;
+    float m = lean_cap ? ref_log2 : -INFINITY, l = 0.f;
 
     auto score = [&](uint32_t raw, int kpos) -> float {
       float s = __uint_as_float(raw) * p.qk_scale;
@@ -400,8 +406,8 @@ attn_extend_kernel(const ExtendParams p) {
           if (lean_cap) {
             const float e0 = fast_exp2(__uint_as_float(v[h][2 * c]) * cap_k1);
             const float e1 = fast_exp2(__uint_as_float(v[h][2 * c + 1]) * cap_k1);
-            p0 = fast_exp2(__fdividef(cap_k2, e0 + 1.0f));
-            p1 = fast_exp2(__fdividef(cap_k2, e1 + 1.0f));
+            p0 = fast_exp2(__fdividef(cap_k2, e0 + 1.0f) + cap_k0);
+            p1 = fast_exp2(__fdividef(cap_k2, e1 + 1.0f) + cap_k0);
             if (edge) {
               const int kp = k0 + h * 32 + 2 * c;
               if (kp > limit || (kp < first && kp >= kept)) p0 = 0.f;
@@ -464,6 +470,21 @@ attn_extend_kernel(const ExtendParams p) {
       uint32_t v[32];
       tc::tmem_ld32(tmem_o + cv * 32, v);
       tc::tmem_ld_wait();
+      if (p.gate && row_ok) {
+        const uint4* grow = reinterpret_cast<const uint4*>(static_cast<const T*>(p.gate) + (q_row0 + tok) * p.gate_stride +
+                                                           static_cast<int64_t>(head_base + r % p.pack) * D + cc * 32);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const uint4 g4 = grow[i];
+          const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 z = unpack2<T>(gw[e]);
+            v[i * 8 + 2 * e] = __float_as_uint(__uint_as_float(v[i * 8 + 2 * e]) * sigmoid_f(z.x));
+            v[i * 8 + 2 * e + 1] = __float_as_uint(__uint_as_float(v[i * 8 + 2 * e + 1]) * sigmoid_f(z.y));
+          }
+        }
+      }
       if (row_ok) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
@@ -521,7 +542,8 @@ static int launch_extend_inst(const ExtendParams& p, int bs, int max_extend_len,
 template <typename T, int D>
 static int launch_extend(const ExtendParams& p, int n_values, int bs, int max_extend_len, cudaStream_t st) {
   // a cap up to 40 keeps e^(-2 cap) a normal fp32 (and 16-bit) number: the one-pass capped form
-  const bool fast = p.logit_cap <= 40.f && p.qk_scale > 0.f && extend_fast_softmax_enabled();
+  const float ref = p.score_bound > 0.f && p.score_bound < p.logit_cap ? p.score_bound : p.logit_cap;
+  const bool fast = ref <= 40.f && p.qk_scale > 0.f && extend_fast_softmax_enabled();
   note_variant("attn_extend d=%d fast_softmax=%d values=%d", D, fast ? 1 : 0, n_values);
   if (n_values == 2)
     return fast ? launch_extend_inst<T, D, true, 2>(p, bs, max_extend_len, st)
@@ -601,8 +623,12 @@ static int extend_heads_impl(const void* q, int64_t q_stride, const void* k_cach
                              const int32_t* extend_start_loc, int bs, int max_extend_len, int Hq, int Hkv,
                              int D, int Dv, float scale, float logit_cap, float out_scale, int causal,
                              int window, int keep_first, const float* sink, int v_head, int n_values,
-                             int64_t o_plane, float* lse, int64_t lse_stride, int dtype, void* stream) {
+                             int64_t o_plane, float* lse, int64_t lse_stride, int dtype, void* stream,
+                             const void* gate = nullptr, int64_t gate_stride = 0, float score_bound = 0.f) {
   using namespace b200;
+  B200_REQUIRE(!gate || (n_values == 1 && gate_stride % 8 == 0 && aligned16(gate)),
+               "b200_attn_extend: the gate rows must be 16-byte aligned (stride %lld)",
+               static_cast<long long>(gate_stride));
   B200_REQUIRE(!lse || (lse_stride >= Hq && !sink), "b200_attn_extend: row sums of %d heads in rows of %lld", Hq,
                static_cast<long long>(lse_stride));
   B200_REQUIRE(keep_first >= 0 && v_head < Hkv, "b200_attn_extend: kept tokens %d, value head %d",
@@ -657,6 +683,9 @@ static int extend_heads_impl(const void* q, int64_t q_stride, const void* k_cach
   p.o_plane = o_plane;
   p.lse = lse;
   p.lse_stride = lse_stride;
+  p.gate = gate;
+  p.gate_stride = gate_stride;
+  p.score_bound = score_bound;
   B200_REQUIRE(bs <= 65535 && Hkv * p.head_tiles <= 65535, "b200_attn_extend: grid too large");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (dtype == B200_BF16)
@@ -680,6 +709,22 @@ int b200_attn_extend_heads(const void* q, int64_t q_stride, const void* k_cache,
                            extend_seq_lens, extend_start_loc, bs, max_extend_len, Hq, Hkv, D, Dv, scale,
                            logit_cap, out_scale, causal, window, keep_first, sink, v_head, n_values, o_plane,
                            nullptr, 0, dtype, stream);
+}
+
+int b200_attn_extend_gated(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
+                           int64_t kv_row_stride, void* o, int64_t o_stride,
+                           const int32_t* req_to_token, int64_t req_to_token_stride,
+                           const int64_t* req_pool_indices, const int64_t* seq_lens,
+                           const int32_t* extend_prefix_lens, const int32_t* extend_seq_lens,
+                           const int32_t* extend_start_loc, int bs, int max_extend_len, int Hq, int Hkv,
+                           int D, int Dv, float scale, float logit_cap, float score_bound, int window,
+                           int keep_first, const float* sink, const void* gate, int64_t gate_stride, int dtype,
+                           void* stream) {
+  return extend_heads_impl(q, q_stride, k_cache, v_cache, kv_row_stride, o, o_stride, req_to_token,
+                           req_to_token_stride, req_pool_indices, seq_lens, extend_prefix_lens,
+                           extend_seq_lens, extend_start_loc, bs, max_extend_len, Hq, Hkv, D, Dv, scale,
+                           logit_cap, 1.f, 1, window, keep_first, sink, -1, 1, 0, nullptr, 0, dtype, stream, gate,
+                           gate_stride, score_bound);
 }
 
 int b200_attn_extend_lse(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,

@@ -178,6 +178,10 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+// tanh(x) = 1 - 2 / (e^(2x) + 1) given x * 2 log2(e): absolute error of a few 1e-7, where the one-instruction
+// approximation below is off by 5e-4
+__device__ __forceinline__ float exact_tanh_log2(float x2) { return 1.0f - __fdividef(2.0f, fast_exp2(x2) + 1.0f); }
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float fast_tanh(float x) {
   float y;
   asm("tanh.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));

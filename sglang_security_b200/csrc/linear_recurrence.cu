@@ -10,6 +10,11 @@
 //             value column that is always 1.  The kernel returns the un-normalised o_t together with
 //             n_t . q_t and m_t per (token, head); the consumer divides by
 //             max(|n_t . q_t|, exp(-m_t)) + den_eps                                          (mLSTM)
+//   channel form : a forget gate per key channel that also decides what is written (HGRN2): with
+//             w = (1 - lower) * sigmoid(-(zf + bias)) per head and channel,
+//             S_t = diag(1 - w_t) S_(t-1) + w_t v_t^T, computed as S += w (v - S): the share that is
+//             forgotten is the share that is written, so the two can not drift apart by rounding; the share w
+//             is formed directly (1 - f would lose its leading digits where f is close to 1).
 //
 // One CTA owns (batch entry, head, a slice of the value columns) and walks the entry's new tokens in
 // order, so a token's result is the same sum in the same order however the sequence was cut into
@@ -75,7 +80,9 @@ __device__ __forceinline__ float log_sigmoid(float z) {
   return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
 }
 
-template <typename T, bool GATES, int kRecRows>
+// FORM 0: decay per head, 1: exponential gates, 2: forget gate per channel (the `k` rows are its
+// pre-activations; `act` then applies to the queries only)
+template <typename T, int FORM, int kRecRows>
 __global__ void __launch_bounds__(kRecMaxThreads)
 linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restrict__ k, int64_t ldk,
                          const T* __restrict__ v, int64_t ldv, const float* __restrict__ gates,
@@ -84,7 +91,9 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
                          const int64_t* __restrict__ slot, const int* __restrict__ tok_pos,
                          const int* __restrict__ ext_start, const int* __restrict__ ext_len,
                          float* __restrict__ out, int64_t ldo, float* __restrict__ aux, int64_t ld_aux,
-                         int H, int D, int E, int P, int CH, int stream_rows) {
+                         int H, int D, int E, int P, int CH, int stream_rows,
+                         const float* __restrict__ f_bias, const float* __restrict__ f_lower) {
+  constexpr bool GATES = FORM == 1;
   extern __shared__ __align__(16) float rec_smem[];
   const int nthreads = blockDim.x, nwarps = nthreads >> 5;
   const int Dp = P * kRecRows;                // padded key size
@@ -131,7 +140,7 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
     s1[2 * a4 + 1] = pack2(v1.y, v1.w);
   }
   float m = (GATES && !fresh) ? st_m[min(cpg, NCP - 1)] : 0.f;
-  const float lam = GATES ? 0.f : decay[h];
+  const float lam = FORM == 0 ? decay[h] : 0.f;
   const int vvalid = max(0, min(ES, E - e0));  // value columns of this slice that exist
   constexpr int PE = 8 / sizeof(T);            // values per 8-byte piece
   auto issue_chunk = [&](int c0, int stage) {
@@ -184,7 +193,12 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
           qv = to_float<T>(stream_rows ? rq[j * D + d] : q[row * ldq + h * D + d]);
           kv = to_float<T>(stream_rows ? rk[j * D + d] : k[row * ldk + h * D + d]);
           qv = rec_act(qv, act) * q_scale;
-          kv = rec_act(kv, act);
+          if (FORM == 2) {                     // the share that is forgotten and written
+            const float z = kv + (f_bias ? f_bias[h * D + d] : 0.f);
+            kv = (1.0f - (f_lower ? f_lower[h * D + d] : 0.f)) / (1.0f + expf(z));
+          } else {
+            kv = rec_act(kv, act);
+          }
         }
         qs[j * Dp + d] = qv;
         ks[j * Dp + d] = kv;
@@ -192,7 +206,7 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
       for (int c = lane; c < ES; c += 32) {
         float x = 0.f;
         if (e0 + c < E)
-          x = rec_act(to_float<T>(stream_rows ? rv[j * ES + c] : v[row * ldv + h * E + e0 + c]), act);
+          x = rec_act(to_float<T>(stream_rows ? rv[j * ES + c] : v[row * ldv + h * E + e0 + c]), FORM == 2 ? 0 : act);
         else if (GATES && e0 + c == E) x = 1.f;
         vs[j * ES + c] = x;
       }
@@ -236,7 +250,7 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
 #pragma unroll 2
     for (int j = 0; j < n; ++j) {
       const float a = GATES ? ga[j] : lam, bb = GATES ? gb[j] : 1.f;
-      const f32x2 a2 = pack2(a, a);
+      const f32x2 a2 = FORM == 2 ? pack2(-1.f, -1.f) : pack2(a, a);
       const float2 vv = *reinterpret_cast<const float2*>(vs + j * ES + 2 * cp);
       const f32x2 ve0 = pack2(vv.x * bb, vv.x * bb), ve1 = pack2(vv.y * bb, vv.y * bb);
       const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(ks + j * Dp) + p;
@@ -245,13 +259,17 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
 #pragma unroll
       for (int r4 = 0; r4 < kRecRows / 4; ++r4) {
         const ulonglong2 kk = k4[r4 * P], qq = q4[r4 * P];     // rows 4 d4 .. 4 d4 + 3 as two row pairs
-        s0[2 * r4] = fma2(a2, s0[2 * r4], mul2(kk.x, ve0));
+        // (channel form: v - S in the place of the product, the share kk in the place of the decay)
+        auto step = [&](f32x2 s, f32x2 kx, f32x2 ve) {
+          return FORM == 2 ? fma2(kx, fma2(a2, s, ve), s) : fma2(a2, s, mul2(kx, ve));
+        };
+        s0[2 * r4] = step(s0[2 * r4], kk.x, ve0);
         acc0a = fma2(s0[2 * r4], qq.x, acc0a);
-        s1[2 * r4] = fma2(a2, s1[2 * r4], mul2(kk.x, ve1));
+        s1[2 * r4] = step(s1[2 * r4], kk.x, ve1);
         acc1a = fma2(s1[2 * r4], qq.x, acc1a);
-        s0[2 * r4 + 1] = fma2(a2, s0[2 * r4 + 1], mul2(kk.y, ve0));
+        s0[2 * r4 + 1] = step(s0[2 * r4 + 1], kk.y, ve0);
         acc0b = fma2(s0[2 * r4 + 1], qq.y, acc0b);
-        s1[2 * r4 + 1] = fma2(a2, s1[2 * r4 + 1], mul2(kk.y, ve1));
+        s1[2 * r4 + 1] = step(s1[2 * r4 + 1], kk.y, ve1);
         acc1b = fma2(s1[2 * r4 + 1], qq.y, acc1b);
       }
       float x0, x1, x2, x3, y0, y1, y2, y3;
@@ -350,18 +368,18 @@ extern "C" int64_t b200_linear_recurrence_state_width(int H, int D, int E, int g
   return static_cast<int64_t>(H) * rec_head_width(D, E, gated);
 }
 
-extern "C" int b200_linear_recurrence(const void* q, int64_t ldq, const void* k, int64_t ldk,
-                                      const void* v, int64_t ldv, const float* gates, int64_t ldg,
-                                      const float* decay, float cap, float q_scale, int act,
-                                      float* state, int64_t ld_state, const int64_t* slot,
-                                      const int* tok_pos, const int* ext_start, const int* ext_len,
-                                      float* out, int64_t ldo, float* aux, int64_t ld_aux, int batch,
-                                      int H, int D, int E, int dtype, void* stream) {
+static int linear_recurrence_impl(const void* q, int64_t ldq, const void* k, int64_t ldk,
+                                  const void* v, int64_t ldv, const float* gates, int64_t ldg,
+                                  const float* decay, const float* f_bias, const float* f_lower, int form,
+                                  float cap, float q_scale, int act, float* state, int64_t ld_state,
+                                  const int64_t* slot, const int* tok_pos, const int* ext_start,
+                                  const int* ext_len, float* out, int64_t ldo, float* aux, int64_t ld_aux,
+                                  int batch, int H, int D, int E, int dtype, void* stream) {
   using namespace b200;
   if (batch == 0) return 0;
   B200_REQUIRE(q && k && v && state && slot && tok_pos && ext_start && ext_len && out,
                "b200_linear_recurrence: null pointer");
-  B200_REQUIRE((gates != nullptr) != (decay != nullptr),
+  B200_REQUIRE(form == 2 || (gates != nullptr) != (decay != nullptr),
                "b200_linear_recurrence: give either gate pre-activations or a decay per head");
   B200_REQUIRE(!gates || aux, "b200_linear_recurrence: the gated form returns (n . q, m) in aux");
   B200_REQUIRE(batch > 0 && H > 0 && D > 0 && E > 0 && D <= kRecMaxRows * 32 && (act == 0 || act == 1),
@@ -400,7 +418,7 @@ extern "C" int b200_linear_recurrence(const void* q, int64_t ldq, const void* k,
   while (CH > 4 && smem_for(CH) > 100 * 1024) CH >>= 1;   // two CTAs per SM
   const size_t smem = smem_for(CH);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  ScopedKernelTimer timer("linear_recurrence", st);
+  ScopedKernelTimer timer(form == 2 ? "channel_recurrence" : "linear_recurrence", st);
   const dim3 grid(ceil_div(ncp, pairs), H, batch);
 #define LAUNCH(TT, G)               \
   do {                              \
@@ -416,12 +434,13 @@ extern "C" int b200_linear_recurrence(const void* q, int64_t ldq, const void* k,
     launch_kernel(kern, grid, dim3(nthreads), smem, st, 1, 0, static_cast<const TT*>(q), ldq,        \
                   static_cast<const TT*>(k), ldk, static_cast<const TT*>(v), ldv, gates, ldg, decay, \
                   cap, q_scale, act, state, ld_state, slot, tok_pos, ext_start, ext_len, out, ldo,   \
-                  aux, ld_aux, H, D, E, P, CH, stream_rows ? 1 : 0);                                 \
+                  aux, ld_aux, H, D, E, P, CH, stream_rows ? 1 : 0, f_bias, f_lower);                \
   } while (0)
 #define BY_G(TT)                  \
   do {                            \
-    if (gates) LAUNCH(TT, true);  \
-    else LAUNCH(TT, false);       \
+    if (form == 2) LAUNCH(TT, 2); \
+    else if (gates) LAUNCH(TT, 1); \
+    else LAUNCH(TT, 0);           \
   } while (0)
   if (dtype == B200_BF16) BY_G(__nv_bfloat16);
   else if (dtype == B200_F16) BY_G(__half);
@@ -430,9 +449,33 @@ extern "C" int b200_linear_recurrence(const void* q, int64_t ldq, const void* k,
 #undef BY_G
 #undef LAUNCH
 #undef LAUNCH_R
-  note_variant("linear_recurrence rows%d threads%d parts%d chunk%d stream%d", kRecRows, nthreads, P, CH, stream_rows ? 1 : 0);
+  note_variant("linear_recurrence form%d rows%d threads%d parts%d chunk%d stream%d", form, kRecRows, nthreads, P, CH, stream_rows ? 1 : 0);
   B200_CHECK_LAUNCH("linear_recurrence_kernel");
   return 0;
+}
+
+extern "C" int b200_linear_recurrence(const void* q, int64_t ldq, const void* k, int64_t ldk,
+                                      const void* v, int64_t ldv, const float* gates, int64_t ldg,
+                                      const float* decay, float cap, float q_scale, int act,
+                                      float* state, int64_t ld_state, const int64_t* slot,
+                                      const int* tok_pos, const int* ext_start, const int* ext_len,
+                                      float* out, int64_t ldo, float* aux, int64_t ld_aux, int batch,
+                                      int H, int D, int E, int dtype, void* stream) {
+  return linear_recurrence_impl(q, ldq, k, ldk, v, ldv, gates, ldg, decay, nullptr, nullptr, gates ? 1 : 0, cap,
+                                q_scale, act, state, ld_state, slot, tok_pos, ext_start, ext_len, out, ldo, aux,
+                                ld_aux, batch, H, D, E, dtype, stream);
+}
+
+// The channel form: zf [T, H * D] are the forget gate's pre-activations, f_bias / f_lower fp32 [H * D] its
+// bias and lower bound (NULL: zero), act 1: silu on the queries.
+extern "C" int b200_channel_recurrence(const void* q, int64_t ldq, const void* zf, int64_t ldf, const void* v,
+                                       int64_t ldv, const float* f_bias, const float* f_lower, float q_scale,
+                                       int act, float* state, int64_t ld_state, const int64_t* slot,
+                                       const int* tok_pos, const int* ext_start, const int* ext_len, float* out,
+                                       int64_t ldo, int batch, int H, int D, int E, int dtype, void* stream) {
+  return linear_recurrence_impl(q, ldq, zf, ldf, v, ldv, nullptr, 0, nullptr, f_bias, f_lower, 2, 0.f, q_scale, act,
+                                state, ld_state, slot, tok_pos, ext_start, ext_len, out, ldo, nullptr, 0, batch,
+                                H, D, E, dtype, stream);
 }
 
 // aux (optional): fp32 [T, 2 H] = (n . q, m) of the gated recurrence; o is divided by

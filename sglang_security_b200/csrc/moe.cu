@@ -4,7 +4,8 @@
 //                      chosen logit, not renormalised; optionally the per-token gate
 //                      sigmoid(w_sg . h) of a shared expert.  One CTA per token.
 //   moe_align        : stable counting sort of the (token, choice) rows by expert -> row offsets per
-//                      expert and the sorted row list.
+//                      expert and the sorted row list; choices with an id past the last expert (identity
+//                      experts) are left out.
 //   moe_grouped_gemm : for every expert, rows[offsets[e] : offsets[e+1]] x W[e]^T with fp32
 //                      accumulation.  GATED: A rows are gathered from the token activations, both
 //                      halves of the fused [gate; up] weight are multiplied in one pass and
@@ -138,18 +139,20 @@ moe_route_kernel(const T* __restrict__ h, int64_t ldh, const float* __restrict__
 // Softmax scores over ALL experts, a choice among groups of neighbouring experts:
 //   s = softmax(z);  choice = s + correction;  a group's score is its largest choice score; only experts
 //   of the `keep` best groups can be chosen (the others count as minus infinity);  the `top` largest choice
-//   scores are taken (ties: lowest index);  weights = s of the chosen / (their sum + 1e-20).
+//   scores are taken (ties: lowest index);  weights = scale * s of the chosen, divided by (their sum +
+//   1e-20) with `renorm`.  Optionally the per-token gate of a shared expert.
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_route_grouped_kernel(const T* __restrict__ h, int64_t ldh, const float* __restrict__ wr,
                          const float* __restrict__ correction, int E, int W, int top, int n_groups,
-                         int keep, int* __restrict__ ids, float* __restrict__ wts) {
+                         int keep, int* __restrict__ ids, float* __restrict__ wts, int renorm, float scale,
+                         const float* __restrict__ wsg, float* __restrict__ gate) {
   __shared__ float z_s[32 * kMaxExpertsPerLane];   // logits, then the scores s
   __shared__ float c_s[32 * kMaxExpertsPerLane];   // choice scores
   __shared__ float g_s[32 * kMaxExpertsPerLane];   // group scores
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  route_logits<T>(h, ldh, wr, nullptr, E, W, nullptr, nullptr, t, z_s);
+  route_logits<T>(h, ldh, wr, nullptr, E, W, wsg, gate, t, z_s);
   __syncthreads();
   if (warp != 0) return;
   float zmax = -INFINITY;
@@ -237,7 +240,7 @@ moe_route_grouped_kernel(const T* __restrict__ h, int64_t ldh, const float* __re
     if (lane == k) mine = sc;
     if (lane == 0) ids[t * top + k] = bi;
   }
-  if (lane < top) wts[t * top + lane] = mine / (wsum + 1e-20f);
+  if (lane < top) wts[t * top + lane] = scale * (renorm ? mine / (wsum + 1e-20f) : mine);
 }
 
 __global__ void __launch_bounds__(1024)
@@ -246,7 +249,10 @@ moe_align_kernel(const int* __restrict__ ids, int N, int E, int* __restrict__ of
   extern __shared__ int cnt[];  // [E + 1]
   for (int e = threadIdx.x; e <= E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < N; i += blockDim.x) atomicAdd(&cnt[ids[i] + 1], 1);
+  for (int i = threadIdx.x; i < N; i += blockDim.x) {
+    const int e = ids[i];
+    if (e < E) atomicAdd(&cnt[e + 1], 1);      // ids past the experts (identity experts) have no matrices
+  }
   __syncthreads();
   if (threadIdx.x == 0)
     for (int e = 0; e < E; ++e) cnt[e + 1] += cnt[e];
@@ -625,6 +631,14 @@ extern "C" int b200_moe_grouped_gemm(const void* a, int64_t lda, const void* w, 
 extern "C" int b200_moe_route_grouped(const void* h, int64_t ldh, const float* wr, const float* correction,
                                       int E, int W, int top, int n_groups, int keep, int* ids, float* wts,
                                       int T, int dtype, void* stream) {
+  return b200_moe_route_softmax(h, ldh, wr, correction, E, W, top, n_groups, keep, 1, 1.0f, nullptr, ids, wts,
+                                nullptr, T, dtype, stream);
+}
+
+extern "C" int b200_moe_route_softmax(const void* h, int64_t ldh, const float* wr, const float* correction,
+                                      int E, int W, int top, int n_groups, int keep, int renorm, float scale,
+                                      const float* wsg, int* ids, float* wts, float* gate, int T, int dtype,
+                                      void* stream) {
   using namespace b200;
   if (T == 0) return 0;
   B200_REQUIRE(h && wr && ids && wts, "b200_moe_route_grouped: null pointer");
@@ -637,7 +651,8 @@ extern "C" int b200_moe_route_grouped(const void* h, int64_t ldh, const float* w
   ScopedKernelTimer timer("moe_route", st);
 #define LAUNCH(TT)                                                                                   \
   launch_kernel(moe_route_grouped_kernel<TT>, dim3(T), dim3(256), 0, st, 1, 0,                      \
-                static_cast<const TT*>(h), ldh, wr, correction, E, W, top, n_groups, keep, ids, wts)
+                static_cast<const TT*>(h), ldh, wr, correction, E, W, top, n_groups, keep, ids, wts,  \
+                renorm, scale, wsg, gate)
   if (dtype == B200_BF16) LAUNCH(__nv_bfloat16);
   else if (dtype == B200_F16) LAUNCH(__half);
   else if (dtype == B200_F32) LAUNCH(float);

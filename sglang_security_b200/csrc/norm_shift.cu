@@ -13,6 +13,12 @@
 //                          in the model dtype, the next sublayer's input; with a second weight the copy is
 //                          the NEXT sublayer's pre-norm instead, x / sqrt(mean(x^2) + eps) * w_next (designs
 //                          with a norm on both sides of every sublayer: one launch per sublayer boundary)
+//   add_normed_mix       : add_normed with every term a mixture-of-experts sublayer and a looped stack need:
+//                          y = sa * a + sb * gb[t] * b + sum_k wts[t, k] * (ids[t, k] < n_experts ?
+//                          rows[t * top + k] : same[t]) — a per-token gate on b, weighted expert rows, identity
+//                          experts that return their input —, then x as above, then x += table[id_t] (a row of
+//                          an embedding table, ahead of the next pass of a loop), then the copy / pre-norm.  16-byte
+//                          loads, y and x stay in registers between the two norms.
 //   softcap_rows         : out = cap * tanh(z / cap) in fp32
 //   scaled_add_layernorm : for designs whose norm sits AFTER the residual sum: y = alpha * x + a + b +
 //                          sum_k wts[t, k] * rows[t * top + k] (terms optional) in fp32, then
@@ -153,42 +159,147 @@ xielu_rows_kernel(const T* __restrict__ z, int64_t ldz, T* __restrict__ out, int
     out[t * ldo + d] = from_float<T>(xielu_exact(to_float<T>(z[t * ldz + d]), pos, neg));
 }
 
-template <typename TA>
+struct AddNormedMix {
+  float* x;
+  int64_t ldx;
+  const void *a, *b, *rows, *same, *table;
+  int64_t lda, ldb, ld_rows, ld_same, ld_table;
+  float sa, sb;
+  const float* gb;           // [T] per-token factor on b, or NULL
+  const float* wts;          // [T, top] or NULL (1)
+  const int* ids;            // [T, top] or NULL (every row is an expert's)
+  int top, n_experts;
+  const int64_t* table_ids;  // [T]
+  const float* w;
+  float eps, mult;
+  void* out_h;
+  int64_t ldh;
+  const float* w_next;
+  int W;
+};
+
+__device__ __forceinline__ float block_sum_any(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
+  __syncthreads();
+  if (l == 0) red[w] = v;
+  __syncthreads();
+  float t = l < nw ? red[l] : 0.f;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+  return t;
+}
+
+// acc[i] += s * p[i] for V consecutive values (V = 1, or one 16-byte load)
+template <typename TA, int V>
+__device__ __forceinline__ void axpy_load(float (&acc)[V], float s, const TA* p) {
+  if constexpr (V == 1) {
+    acc[0] = fmaf(s, to_float<TA>(*p), acc[0]);
+  } else {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const TA* e = reinterpret_cast<const TA*>(&u);
+#pragma unroll
+    for (int i = 0; i < V; ++i) acc[i] = fmaf(s, to_float<TA>(e[i]), acc[i]);
+  }
+}
+
+// A thread owns NC chunks of V consecutive coordinates of one token's row.
+template <typename TA, int V, int NC>
 __global__ void __launch_bounds__(kRowThreads)
-add_normed_kernel(float* __restrict__ x, int64_t ldx, const TA* __restrict__ a, int64_t lda, float sa,
-                  const TA* __restrict__ b, int64_t ldb, float sb, const TA* __restrict__ y,
-                  int64_t ldy, int top, const float* __restrict__ w, float eps, float mult,
-                  TA* __restrict__ out_h, int64_t ldh, int W, const float* __restrict__ w_next) {
+add_normed_mix_kernel(const AddNormedMix p) {
   __shared__ float red[kRowThreads / 32];
-  const int t = blockIdx.x;
-  auto term = [&](int d) {
-    float v = 0.f;
-    if (a) v = sa * to_float<TA>(a[t * lda + d]);
-    if (b) v = fmaf(sb, to_float<TA>(b[t * ldb + d]), v);
-    if (y)
-      for (int k = 0; k < top; ++k) v += to_float<TA>(y[(static_cast<int64_t>(t) * top + k) * ldy + d]);
-    return v;
-  };
+  const int64_t t = blockIdx.x;
+  const int W = p.W;
+  float y[NC][V];
   float s = 0.f;
-  for (int d = threadIdx.x; d < W; d += kRowThreads) {
-    const float v = term(d);
-    s = fmaf(v, v, s);
+  const float gb = p.b ? (p.gb ? p.gb[t] : 1.f) * p.sb : 0.f;
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int d = (c * blockDim.x + threadIdx.x) * V;
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[c][i] = 0.f;
+    if (d < W) {
+      if (p.a) axpy_load<TA, V>(y[c], p.sa, static_cast<const TA*>(p.a) + t * p.lda + d);
+      if (p.b) axpy_load<TA, V>(y[c], gb, static_cast<const TA*>(p.b) + t * p.ldb + d);
+      if (p.rows || p.ids) {
+#pragma unroll 4
+        for (int k = 0; k < p.top; ++k) {
+          const float wk = p.wts ? p.wts[t * p.top + k] : 1.f;
+          const bool own = p.ids && p.ids[t * p.top + k] >= p.n_experts;
+          axpy_load<TA, V>(y[c], wk, own ? static_cast<const TA*>(p.same) + t * p.ld_same + d
+                                         : static_cast<const TA*>(p.rows) + (t * p.top + k) * p.ld_rows + d);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) s = fmaf(y[c][i], y[c][i], s);
+    }
   }
-  s = block_sum(s, red);
-  const float r = mult / sqrtf(s / static_cast<float>(W) + eps);
+  s = block_sum_any(s, red);
+  const float r = p.mult / sqrtf(s / static_cast<float>(W) + p.eps);
   float s2 = 0.f;
-  for (int d = threadIdx.x; d < W; d += kRowThreads) {
-    const float nx = fmaf(term(d) * r, w ? w[d] : 1.f, x[t * ldx + d]);
-    x[t * ldx + d] = nx;
-    s2 = fmaf(nx, nx, s2);
-    if (out_h && !w_next) out_h[t * ldh + d] = from_float<TA>(nx);
+  const TA* extra = p.table ? static_cast<const TA*>(p.table) + p.table_ids[t] * p.ld_table : nullptr;
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int d = (c * blockDim.x + threadIdx.x) * V;
+    if (d < W) {
+      float* xr = p.x + t * p.ldx + d;
+      float nx[V];
+      if constexpr (V == 1) {
+        nx[0] = fmaf(y[c][0] * r, p.w ? p.w[d] : 1.f, xr[0]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+          const float4 xv = *reinterpret_cast<const float4*>(xr + i);
+          const float4 wv = p.w ? *reinterpret_cast<const float4*>(p.w + d + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+          nx[i] = fmaf(y[c][i] * r, wv.x, xv.x);
+          nx[i + 1] = fmaf(y[c][i + 1] * r, wv.y, xv.y);
+          nx[i + 2] = fmaf(y[c][i + 2] * r, wv.z, xv.z);
+          nx[i + 3] = fmaf(y[c][i + 3] * r, wv.w, xv.w);
+        }
+      }
+      if (extra) axpy_load<TA, V>(nx, 1.f, extra + d);
+      if constexpr (V == 1) {
+        xr[0] = nx[0];
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; i += 4)
+          *reinterpret_cast<float4*>(xr + i) = make_float4(nx[i], nx[i + 1], nx[i + 2], nx[i + 3]);
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        s2 = fmaf(nx[i], nx[i], s2);
+        y[c][i] = nx[i];
+      }
+    }
   }
-  if (!out_h || !w_next) return;
-  // the next sublayer's pre-norm of the new residual (each thread re-reads the elements it wrote)
-  s2 = block_sum(s2, red);
-  const float r2 = 1.0f / sqrtf(s2 / static_cast<float>(W) + eps);
-  for (int d = threadIdx.x; d < W; d += kRowThreads)
-    out_h[t * ldh + d] = from_float<TA>(x[t * ldx + d] * r2 * w_next[d]);
+  if (!p.out_h) return;
+  float r2 = 1.f;
+  if (p.w_next) {
+    s2 = block_sum_any(s2, red);
+    r2 = 1.0f / sqrtf(s2 / static_cast<float>(W) + p.eps);
+  }
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int d = (c * blockDim.x + threadIdx.x) * V;
+    if (d >= W) continue;
+    TA* dst = static_cast<TA*>(p.out_h) + t * p.ldh + d;
+    if constexpr (V == 1) {
+      dst[0] = from_float<TA>(y[c][0] * r2 * (p.w_next ? p.w_next[d] : 1.f));
+    } else {
+      uint4 u;
+      TA* e = reinterpret_cast<TA*>(&u);
+#pragma unroll
+      for (int i = 0; i < V; i += 4) {
+        const float4 wv = p.w_next ? *reinterpret_cast<const float4*>(p.w_next + d + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+        e[i] = from_float<TA>(y[c][i] * r2 * wv.x);
+        e[i + 1] = from_float<TA>(y[c][i + 1] * r2 * wv.y);
+        e[i + 2] = from_float<TA>(y[c][i + 2] * r2 * wv.z);
+        e[i + 3] = from_float<TA>(y[c][i + 3] * r2 * wv.w);
+      }
+      *reinterpret_cast<uint4*>(dst) = u;
+    }
+  }
 }
 
 template <typename T>
@@ -327,25 +438,8 @@ extern "C" int b200_add_normed_next(float* x, int64_t ldx, const void* a, int64_
                                     int64_t ld_rows, int top, const float* w, float eps, float mult,
                                     void* out_h, int64_t ldh, const float* w_next, int T, int W,
                                     int dtype, void* stream) {
-  using namespace b200;
-  if (T == 0) return 0;
-  B200_REQUIRE(x && (a || b || rows) && T > 0 && W > 0, "b200_add_normed: bad arguments");
-  B200_REQUIRE(!rows || top > 0, "b200_add_normed: rows without a count per token");
-  B200_REQUIRE(!w_next || out_h, "b200_add_normed: a next norm without an output");
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  ScopedKernelTimer timer("add_normed", st);
-#define LAUNCH(TA)                                                                                   \
-  launch_kernel(add_normed_kernel<TA>, dim3(T), dim3(kRowThreads), 0, st, 1, 0, x, ldx,             \
-                static_cast<const TA*>(a), lda, sa, static_cast<const TA*>(b), ldb, sb,              \
-                static_cast<const TA*>(rows), ld_rows, top, w, eps, mult, static_cast<TA*>(out_h),   \
-                ldh, W, w_next)
-  if (dtype == B200_BF16) LAUNCH(__nv_bfloat16);
-  else if (dtype == B200_F16) LAUNCH(__half);
-  else if (dtype == B200_F32) LAUNCH(float);
-  else B200_REQUIRE(false, "b200_add_normed: dtype %d", dtype);
-#undef LAUNCH
-  B200_CHECK_LAUNCH("add_normed_kernel");
-  return 0;
+  return b200_add_normed_mix(x, ldx, a, lda, sa, b, ldb, sb, nullptr, rows, ld_rows, nullptr, nullptr, top, 0,
+                             nullptr, 0, w, eps, mult, nullptr, 0, nullptr, out_h, ldh, w_next, T, W, dtype, stream);
 }
 
 extern "C" int b200_add_normed(float* x, int64_t ldx, const void* a, int64_t lda, float sa,
@@ -354,6 +448,57 @@ extern "C" int b200_add_normed(float* x, int64_t ldx, const void* a, int64_t lda
                                int T, int W, int dtype, void* stream) {
   return b200_add_normed_next(x, ldx, a, lda, sa, b, ldb, sb, rows, ld_rows, top, w, eps, mult, out_h,
                               ldh, nullptr, T, W, dtype, stream);
+}
+
+extern "C" int b200_add_normed_mix(float* x, int64_t ldx, const void* a, int64_t lda, float sa, const void* b,
+                                   int64_t ldb, float sb, const float* gb, const void* rows, int64_t ld_rows,
+                                   const float* wts, const int* ids, int top, int n_experts, const void* same,
+                                   int64_t ld_same, const float* w, float eps, float mult, const void* table,
+                                   int64_t ld_table, const int64_t* table_ids, void* out_h, int64_t ldh,
+                                   const float* w_next, int T, int W, int dtype, void* stream) {
+  using namespace b200;
+  if (T == 0) return 0;
+  B200_REQUIRE(x && (a || b || rows) && T > 0 && W > 0, "b200_add_normed_mix: bad arguments");
+  B200_REQUIRE((!rows && !ids) || top > 0, "b200_add_normed_mix: rows without a count per token");
+  B200_REQUIRE(!ids || (rows && same), "b200_add_normed_mix: expert ids need the expert rows and the identity rows");
+  B200_REQUIRE(!w_next || out_h, "b200_add_normed_mix: a next norm without an output");
+  B200_REQUIRE(!table || table_ids, "b200_add_normed_mix: a table without row ids");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  ScopedKernelTimer timer("add_normed", st);
+  const AddNormedMix p{x, ldx, a, b, rows, same, table, lda, ldb, ld_rows, ld_same, ld_table, sa, sb, gb, wts, ids, top,
+                       n_experts, table_ids, w, eps, mult, out_h, ldh, w_next, W};
+  // one 16-byte chunk per thread and pass when every row allows it
+  const int v = dtype == B200_F32 ? 4 : 8;
+  auto fits = [&](const void* q, int64_t ld) { return !q || (aligned16(q) && ld % v == 0); };
+  const bool vec = W % v == 0 && aligned16(x) && ldx % 4 == 0 && fits(a, lda) && fits(b, ldb) && fits(rows, ld_rows) &&
+                   fits(same, ld_same) && fits(table, ld_table) && fits(out_h, ldh) && aligned16(w) && aligned16(w_next) &&
+                   W <= v * kRowThreads * 4;
+  const int chunks = vec ? W / v : W;
+  int nc = 1;
+  while (nc * kRowThreads < chunks) nc <<= 1;
+  B200_REQUIRE(nc <= 32, "b200_add_normed_mix: width %d too large for unaligned rows", W);
+  int nt = min(kRowThreads, ceil_div(ceil_div(chunks, nc), 32) * 32);
+#define LAUNCH(TA, V, NC) launch_kernel(add_normed_mix_kernel<TA, V, NC>, dim3(T), dim3(nt), 0, st, 1, 0, p)
+#define BY_NC(TA, V)                                                                                 \
+  do {                                                                                               \
+    if (vec) {                                                                                       \
+      if (nc == 1) LAUNCH(TA, V, 1);                                                                 \
+      else if (nc == 2) LAUNCH(TA, V, 2);                                                            \
+      else LAUNCH(TA, V, 4);                                                                         \
+    } else if (nc <= 4) {                                                                            \
+      LAUNCH(TA, 1, 4);                                                                              \
+    } else {                                                                                         \
+      LAUNCH(TA, 1, 32);                                                                             \
+    }                                                                                                \
+  } while (0)
+  if (dtype == B200_BF16) BY_NC(__nv_bfloat16, 8);
+  else if (dtype == B200_F16) BY_NC(__half, 8);
+  else if (dtype == B200_F32) BY_NC(float, 4);
+  else B200_REQUIRE(false, "b200_add_normed_mix: dtype %d", dtype);
+#undef BY_NC
+#undef LAUNCH
+  B200_CHECK_LAUNCH("add_normed_mix_kernel");
+  return 0;
 }
 
 extern "C" int b200_softcap_rows(const void* z, int64_t ldz, float* out, int64_t ldo, int T, int V,

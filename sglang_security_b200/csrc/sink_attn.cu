@@ -11,6 +11,7 @@
 //   * RMS norm of each value head (no weight), and a mix of the normed values with the values another
 //     layer cached for the same token: v <- (1 - lambda) v + lambda v_first;
 //   * a soft cap on the scaled scores: s <- cap * tanh(s / cap);
+//   * an element-wise output gate: the heads' outputs are multiplied by sigmoid(gate[t, h, e]);
 //   * the weights of every query head applied to the values of EVERY key/value head (one grid plane
 //     per value head), for designs that mix the heads' weights after the softmax: the mixed output is
 //     a linear combination of these per-head products (csrc/head_mix.cu).
@@ -61,7 +62,22 @@ __device__ __forceinline__ float normed(const T* row, int idx, const float* w, c
 
 template <typename T>
 __device__ void group_inv_rms(const T* row, int n, int group, float eps, float* inv, float* red) {
-  // few groups (the whole projection, or one per head): one block-wide sum per group
+  if (group <= 512 && n > group) {             // one group per head: a warp each
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int g = warp; g * group < n; g += kPrepThreads / 32) {
+      float s = 0.f;
+      for (int d = lane; d < group; d += 32) {
+        const float x = to_float<T>(row[g * group + d]);
+        s = fmaf(x, x, s);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      if (lane == 0) inv[g] = 1.0f / sqrtf(s / static_cast<float>(group) + eps);
+    }
+    __syncthreads();
+    return;
+  }
+  // few groups (the whole projection): one block-wide sum per group
   for (int g = 0; g * group < n; ++g) {
     float s = 0.f;
     for (int d = threadIdx.x; d < group; d += kPrepThreads) {
@@ -176,7 +192,8 @@ sink_attn_kernel(const float* __restrict__ q, int64_t ldq, const TP* __restrict_
                  int64_t ld_r2t, const int64_t* __restrict__ req_idx, const int* __restrict__ tok_pos,
                  const int* __restrict__ tok_b, const float* __restrict__ sink, float scale, int window,
                  int keep_first, TO* __restrict__ out, int64_t ldo, int H, int G, int D, int E,
-                 const int* __restrict__ tok_list, float softcap, int64_t ldo_plane) {
+                 const int* __restrict__ tok_list, float softcap, int64_t ldo_plane,
+                 const TP* __restrict__ gate, int64_t ld_gate) {
   extern __shared__ __align__(16) float sink_smem[];
   constexpr int RH = kSinkHeads;
   const int nw = blockDim.x >> 5;
@@ -378,7 +395,9 @@ sink_attn_kernel(const float* __restrict__ q, int64_t ldq, const TP* __restrict_
       const int r = i / E, e = i - r * E;
       float o = 0.f;
       for (int w = 0; w < nw; ++w) o = fmaf(wacc[(w * RH + r) * E + e], wf[w * RH + r], o);
-      out[t * ldo + (hb + r) * E + e] = from_float<TO>(o / wt[r]);
+      o /= wt[r];
+      if (gate) o *= sigmoid_f(to_float<TP>(gate[t * ld_gate + (hb + r) * E + e]));
+      out[t * ldo + (hb + r) * E + e] = from_float<TO>(o);
     }
   }
 }
@@ -442,6 +461,15 @@ extern "C" int b200_qk_norm_rope_write(const void* q, int64_t ldq, const void* k
                              ldqo16, T, H, G, D, E, 0.f, 0, 0, nullptr, nullptr, 0, 0, dtype, stream);
 }
 
+static int sink_attn_impl(const float* q, int64_t ldq, const void* pool, int64_t ld_pool,
+                          int k_off, int v_off, const int* req_to_token, int64_t ld_r2t,
+                          const int64_t* req_idx, const int* tok_pos, const int* tok_b,
+                          const float* sink, float scale, float softcap, int window,
+                          int keep_first, void* out, int64_t ldo, int all_values,
+                          int64_t ldo_plane, int T, int H, int G, int D, int E,
+                          const int* tok_list, int max_keys, const void* gate, int64_t ld_gate, int dtype,
+                          void* stream);
+
 // softcap > 0: scores are capped (cap * tanh(s / cap)) before the softmax.  all_values != 0: the weights
 // of every query head are applied to the values of every key/value head; `out` is then fp32
 // [G planes][T rows of ldo][H, E] with `ldo_plane` elements between planes.
@@ -452,6 +480,32 @@ extern "C" int b200_sink_attn_heads(const float* q, int64_t ldq, const void* poo
                                     int keep_first, void* out, int64_t ldo, int all_values,
                                     int64_t ldo_plane, int T, int H, int G, int D, int E,
                                     const int* tok_list, int max_keys, int dtype, void* stream) {
+  return sink_attn_impl(q, ldq, pool, ld_pool, k_off, v_off, req_to_token, ld_r2t, req_idx, tok_pos, tok_b, sink,
+                        scale, softcap, window, keep_first, out, ldo, all_values, ldo_plane, T, H, G, D, E,
+                        tok_list, max_keys, nullptr, 0, dtype, stream);
+}
+
+// gate (optional, [T rows of ld_gate][H, E] in the pool's dtype): the output is multiplied by its sigmoid
+extern "C" int b200_sink_attn_gated(const float* q, int64_t ldq, const void* pool, int64_t ld_pool, int k_off,
+                                    int v_off, const int* req_to_token, int64_t ld_r2t,
+                                    const int64_t* req_idx, const int* tok_pos, const int* tok_b,
+                                    const float* sink, float scale, float softcap, int window, int keep_first,
+                                    const void* gate, int64_t ld_gate, void* out, int64_t ldo, int T, int H,
+                                    int G, int D, int E, const int* tok_list, int max_keys, int dtype,
+                                    void* stream) {
+  return sink_attn_impl(q, ldq, pool, ld_pool, k_off, v_off, req_to_token, ld_r2t, req_idx, tok_pos, tok_b, sink,
+                        scale, softcap, window, keep_first, out, ldo, 0, 0, T, H, G, D, E, tok_list, max_keys, gate,
+                        ld_gate, dtype, stream);
+}
+
+static int sink_attn_impl(const float* q, int64_t ldq, const void* pool, int64_t ld_pool,
+                          int k_off, int v_off, const int* req_to_token, int64_t ld_r2t,
+                          const int64_t* req_idx, const int* tok_pos, const int* tok_b,
+                          const float* sink, float scale, float softcap, int window,
+                          int keep_first, void* out, int64_t ldo, int all_values,
+                          int64_t ldo_plane, int T, int H, int G, int D, int E,
+                          const int* tok_list, int max_keys, const void* gate, int64_t ld_gate, int dtype,
+                          void* stream) {
   using namespace b200;
   if (T == 0) return 0;
   B200_REQUIRE(q && pool && req_to_token && req_idx && tok_pos && tok_b && out,
@@ -478,7 +532,7 @@ extern "C" int b200_sink_attn_heads(const float* q, int64_t ldq, const void* poo
   launch_kernel(sink_attn_kernel<TT, TO>, grid, dim3(nw * 32), smem, st, 1, 0, q, ldq,               \
                 static_cast<const TT*>(pool), ld_pool, k_off, v_off, req_to_token, ld_r2t, req_idx,  \
                 tok_pos, tok_b, sink, scale, window, keep_first, static_cast<TO*>(out), ldo, H, G, D, \
-                E, tok_list, softcap, ldo_plane)
+                E, tok_list, softcap, ldo_plane, static_cast<const TT*>(gate), ld_gate)
   if (all_values) {
     if (dtype == B200_BF16) LAUNCH(__nv_bfloat16, float);
     else if (dtype == B200_F16) LAUNCH(__half, float);

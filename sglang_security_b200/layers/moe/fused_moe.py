@@ -6,7 +6,9 @@
     GroupedSoftmaxRouter : z = W_r h in fp32; scores s = softmax(z) over ALL experts; the choice is made
                    on s + correction, among the experts of the `keep` groups (of `groups` equal groups
                    of neighbours) whose best choice score is largest; weights = the chosen experts' s,
-                   divided by their sum (+ 1e-20).
+                   divided by their sum (+ 1e-20) or, renormalize=False, as they are, times `scale`.
+                   The last `identity` of the scored experts have no matrices: their output is the
+                   sublayer's input.  Optionally the scalar gate of a shared expert.
     FusedExperts : all experts' gated feed-forwards W_down (act(W_gate h) * (W_up h)) as two grouped
                    GEMMs over the (token, choice) rows sorted by expert; nothing is read back to the
                    host, so the step stays capturable.  Returns one row per (token, choice); the
@@ -60,28 +62,39 @@ class TopKRouter(nn.Module):
 
 class GroupedSoftmaxRouter(nn.Module):
     def __init__(self, width: int, experts: int, top: int, groups: int = 1, keep: int = 1,
-                 correction: bool = True):
+                 correction: bool = True, identity: int = 0, renormalize: bool = True, scale: float = 1.0,
+                 shared_gate: bool = False):
         super().__init__()
-        if experts % groups or not 0 < keep <= groups or keep * (experts // groups) < top:
+        experts += identity                          # all that are scored
+        if experts % groups or not 0 < keep <= groups or not 0 < top <= keep * (experts // groups):
             raise ValueError(f"{experts} experts in {groups} groups, {keep} kept, top {top}")
         self.experts, self.top, self.groups, self.keep = experts, top, groups, keep
+        self.identity, self.renormalize, self.scale = identity, bool(renormalize), float(scale)
+        self.shared_gate = (nn.Parameter(torch.zeros(width, dtype=torch.float32), requires_grad=False)
+                            if shared_gate else None)
         self.weight = nn.Parameter(torch.zeros(experts, width, dtype=torch.float32), requires_grad=False)
         self.correction = (nn.Parameter(torch.zeros(experts, dtype=torch.float32), requires_grad=False)
                            if correction else None)
 
     def forward(self, h: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
         """h [T, width] (fp32 or the model dtype) -> (ids int32 [T, top], weights fp32 [T, top])."""
+        return self.route(h)[:2]
+
+    def route(self, h: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
+        """-> (ids, weights, the shared expert's gate fp32 [T] or None); ids of identity experts are the last."""
         if not h.is_cuda:
             raise _lib.B200Error("GroupedSoftmaxRouter: tensor must live on a CUDA device (no CPU path)")
         t, w = h.shape
         ids = torch.empty((t, self.top), dtype=torch.int32, device=h.device)
         wts = torch.empty((t, self.top), dtype=torch.float32, device=h.device)
-        rc = _lib.load().b200_moe_route_grouped(
+        gate = torch.empty((t,), dtype=torch.float32, device=h.device) if self.shared_gate is not None else None
+        rc = _lib.load().b200_moe_route_softmax(
             h.data_ptr(), h.stride(0), self.weight.data_ptr(), _lib.ptr(self.correction), self.experts, w,
-            self.top, self.groups, self.keep, ids.data_ptr(), wts.data_ptr(), t, _lib.dtype_code(h.dtype),
-            _lib.current_stream())
-        _lib.check(rc, "b200_moe_route_grouped")
-        return ids, wts
+            self.top, self.groups, self.keep, 1 if self.renormalize else 0, self.scale,
+            _lib.ptr(self.shared_gate), ids.data_ptr(), wts.data_ptr(), _lib.ptr(gate), t,
+            _lib.dtype_code(h.dtype), _lib.current_stream())
+        _lib.check(rc, "b200_moe_route_softmax")
+        return ids, wts, gate
 
 
 class FusedExperts(nn.Module):
@@ -99,7 +112,8 @@ class FusedExperts(nn.Module):
         self.w_down.data[e].copy_(down)
 
     def forward(self, h: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
-        """h [T, width], ids [T, top] -> expert outputs [T * top, width] (row t * top + k)."""
+        """h [T, width], ids [T, top] -> expert outputs [T * top, width] (row t * top + k).  Rows of ids past
+        the last expert (identity experts) are not written."""
         t, top = ids.shape
         n = t * top
         lib, st, code = _lib.load(), _lib.current_stream(), _lib.dtype_code(h.dtype)

@@ -13,6 +13,10 @@ the sequence was cut.  Two mixers are built on it:
                             a weight over all heads, an output gate sigmoid(W_g h), W_o
     DecayedLinearAttention  constant decay per head, silu on q, k and v, RMS norm over all heads
                             together with a weight, an output gate, W_o
+    ChannelForgetMixer      a forget gate per head and channel between a lower bound and 1 that also decides
+                            what is written (Qin et al., "HGRN2: Gated Linear RNNs with State Expansion"):
+                            f = l + (1 - l) sigmoid(W_f h + b), S = diag(f) S + (1 - f) v^T, o = S^T silu(W_q h),
+                            RMS norm per head with one weight shared by the heads, W_o
 """
 from __future__ import annotations
 
@@ -86,6 +90,30 @@ def gated_group_rmsnorm(o: torch.Tensor, weight: Optional[torch.Tensor], z: Opti
     return out
 
 
+def channel_recurrence(q: torch.Tensor, zf: torch.Tensor, v: torch.Tensor, bias: Optional[torch.Tensor],
+                       lower: Optional[torch.Tensor], heads: int, dim: int, vdim: int, state: torch.Tensor,
+                       fb, q_scale: float = 1.0, silu: bool = True) -> torch.Tensor:
+    """q, zf [T, heads * dim] (zf: the forget gates' pre-activations), v [T, heads * vdim], row-strided views
+    of one dtype; bias, lower fp32 [heads * dim] -> fp32 [T, heads * vdim].  silu applies to q."""
+    if not q.is_cuda:
+        raise _lib.B200Error("channel_recurrence: tensors must live on a CUDA device (no CPU path)")
+    for t in (q, zf, v):
+        if t.stride(-1) != 1 or t.dtype != q.dtype:
+            raise _lib.B200Error("channel_recurrence: q, zf, v need contiguous rows of one dtype")
+    for t in (bias, lower):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != heads * dim or not t.is_contiguous()):
+            raise _lib.B200Error("channel_recurrence: bias and lower bound are fp32 [heads * dim]")
+    out = torch.empty((q.shape[0], heads * vdim), dtype=torch.float32, device=q.device)
+    rc = _lib.load().b200_channel_recurrence(
+        q.data_ptr(), q.stride(0), zf.data_ptr(), zf.stride(0), v.data_ptr(), v.stride(0), _lib.ptr(bias),
+        _lib.ptr(lower), float(q_scale), 1 if silu else 0, state.data_ptr(), state.stride(0),
+        fb.req_pool_indices.data_ptr(), fb.tok_pos.data_ptr(), fb.ext_start.data_ptr(), fb.ext_len.data_ptr(),
+        out.data_ptr(), out.stride(0), int(fb.batch_size), heads, dim, vdim, _lib.dtype_code(q.dtype),
+        _lib.current_stream())
+    _lib.check(rc, "b200_channel_recurrence")
+    return out
+
+
 class _MatrixMemoryMixer(nn.Module):
     """Shared plumbing: one fused projection [q ; k ; v ; g], the output norm weight and W_o."""
 
@@ -154,4 +182,41 @@ class DecayedLinearAttention(_MatrixMemoryMixer):
                               decay=self.decay, silu=True)
         y = gated_group_rmsnorm(o, self.norm_weight, g, self.heads * self.vdim, self.eps, self.params_dtype)
         out, _ = self.o_proj(y)
+        return out
+
+
+class ChannelForgetMixer(nn.Module):
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, layer_id: int, eps: float,
+                 params_dtype: torch.dtype = torch.bfloat16):
+        super().__init__()
+        self.width, self.heads, self.dim, self.vdim = width, heads, dim, vdim
+        self.layer_id, self.eps, self.params_dtype = layer_id, float(eps), params_dtype
+        kw = dict(bias=False, params_dtype=params_dtype, tp_rank=0, tp_size=1)
+        self.sizes = [heads * dim, heads * dim, heads * vdim]          # one input GEMM: [q ; f ; v]
+        self.qfv_proj = ColumnParallelLinear(width, sum(self.sizes), **kw)
+        self.o_proj = RowParallelLinear(heads * vdim, width, **kw)
+        f32 = dict(dtype=torch.float32)
+        self.f_bias = nn.Parameter(torch.zeros(heads * dim, **f32), requires_grad=False)
+        self.f_lower = nn.Parameter(torch.zeros(heads * dim, **f32), requires_grad=False)
+        # the output norm's weight [vdim] is shared by the heads: stored once per head
+        self.norm_weight = nn.Parameter(torch.ones(heads * vdim, **f32), requires_grad=False)
+
+    def state_width(self) -> int:
+        return state_width(self.heads, self.dim, self.vdim, False)
+
+    def load_part(self, which: str, w: torch.Tensor) -> None:
+        i = "qfv".index(which)
+        lo = sum(self.sizes[:i])
+        self.qfv_proj.weight.data[lo:lo + self.sizes[i]].copy_(w)
+
+    def forward(self, h: torch.Tensor, fb, cache_id: Optional[int] = None) -> torch.Tensor:
+        """cache_id: the state this run of the layer carries, where it is not the layer's own (a looped
+        layer has one per pass)."""
+        y, _ = self.qfv_proj(h)
+        a = self.sizes
+        q, zf, v = y[:, :a[0]], y[:, a[0]:a[0] + a[1]], y[:, a[0] + a[1]:]
+        state = fb.state_pool.get(self.layer_id if cache_id is None else cache_id)
+        o = channel_recurrence(q, zf, v, self.f_bias, self.f_lower, self.heads, self.dim, self.vdim, state, fb)
+        z = gated_group_rmsnorm(o, self.norm_weight, None, self.vdim, self.eps, self.params_dtype)
+        out, _ = self.o_proj(z)
         return out

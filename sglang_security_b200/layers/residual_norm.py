@@ -1,20 +1,22 @@
 """Norm on a sublayer's OUTPUT followed by the residual add, for designs whose sublayers read the
 32-bit residual itself (csrc/norm_shift.cu add_normed):
 
-    y = sa * a + sb * b + sum_k rows[t * top + k]        (fp32 sum of the terms given)
+    y = sa * a + sb * gate[t] * b + sum_k w[t, k] * rows[t * top + k]        (fp32 sum of the terms given)
     x += mult * y / sqrt(mean(y^2) + eps) * weight
+    x += table[id_t]                                     (on request: ahead of the next pass of a loop)
 
 `AddNormed` owns the weight; one launch does the sum, the norm, the add and, on request, the copy of
 the new residual in the model dtype that the next sublayer's matrix products read.  For designs with a
 norm BEFORE every sublayer as well, that copy is the next sublayer's pre-norm
-x / sqrt(mean(x^2) + eps) * next_weight instead (still the one launch).  `ResidualRMSNorm`
+x / sqrt(mean(x^2) + eps) * next_weight instead (still the one launch).  Choices of an identity expert
+(ids past the last expert) add the sublayer's input instead of an expert row.  `ResidualRMSNorm`
 is the plain RMS norm of the fp32 residual with a per-coordinate weight (a model's final norm), its
 output in the model dtype.  `PostSumLayerNorm` is for designs whose norm follows the residual SUM:
 x <- LN(alpha * x + terms) with weight and bias (csrc/norm_shift.cu scaled_add_layernorm), the expert
 rows weighted inside the same fp32 sum; without terms it is a plain layer norm of the residual.  `softcap` is the logit cap cap * tanh(z / cap) with a fp32 result."""
 from __future__ import annotations
 
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -31,9 +33,15 @@ class AddNormed(nn.Module):
     def forward(self, x: torch.Tensor, a: Optional[torch.Tensor] = None, sa: float = 1.0,
                 b: Optional[torch.Tensor] = None, sb: float = 1.0, rows: Optional[torch.Tensor] = None,
                 top: int = 0, out_dtype: Optional[torch.dtype] = None,
-                next_weight: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                next_weight: Optional[torch.Tensor] = None, b_gate: Optional[torch.Tensor] = None,
+                row_weights: Optional[torch.Tensor] = None, row_ids: Optional[torch.Tensor] = None,
+                experts: int = 0, same: Optional[torch.Tensor] = None,
+                inject: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> Optional[torch.Tensor]:
         """x: fp32 residual [T, W], updated in place.  -> the new x in `out_dtype` (None: not asked), or
-        with `next_weight` (fp32 [W]) its RMS norm times that weight."""
+        with `next_weight` (fp32 [W]) its RMS norm times that weight.  b_gate: fp32 [T], a factor on b per
+        token; row_weights: fp32 [T, top]; row_ids: int32 [T, top] with `experts` and `same` [T, W]: choices
+        with an id of at least `experts` add `same`; inject: (table, int64 row ids [T]) added to x after the
+        sum."""
         if not x.is_cuda:
             raise _lib.B200Error("AddNormed: tensor must live on a CUDA device (no CPU path)")
         if x.dtype != torch.float32 or x.dim() != 2 or x.stride(1) != 1:
@@ -42,21 +50,29 @@ class AddNormed(nn.Module):
         if not terms:
             raise _lib.B200Error("AddNormed: nothing to add")
         dt = terms[0].dtype
-        for v in terms:
+        table, table_ids = inject if inject is not None else (None, None)
+        for v in terms + [v for v in (same, table) if v is not None]:
             if v.dtype != dt or v.stride(-1) != 1:
                 raise _lib.B200Error("AddNormed: terms must share a dtype and have contiguous rows")
         t, w = x.shape
+        for v, shape in ((b_gate, (t,)), (row_weights, (t, top))):
+            if v is not None and (v.dtype != torch.float32 or tuple(v.shape) != shape or not v.is_contiguous()):
+                raise _lib.B200Error(f"AddNormed: fp32 factors of shape {shape} are expected")
+        if row_ids is not None and (row_ids.dtype != torch.int32 or tuple(row_ids.shape) != (t, top)
+                                    or not row_ids.is_contiguous() or same is None):
+            raise _lib.B200Error("AddNormed: expert ids are int32 [T, top] and come with the identity rows")
         out = None
         if out_dtype is not None and (out_dtype != torch.float32 or next_weight is not None):
             if out_dtype != dt:
                 raise _lib.B200Error("AddNormed: the copy of the residual has the terms' dtype")
             out = torch.empty((t, w), dtype=out_dtype, device=x.device)
         ld = lambda v: v.stride(0) if v is not None else 0
-        rc = _lib.load().b200_add_normed_next(
+        rc = _lib.load().b200_add_normed_mix(
             x.data_ptr(), x.stride(0), _lib.ptr(a), ld(a), float(sa), _lib.ptr(b), ld(b), float(sb),
-            _lib.ptr(rows), ld(rows), int(top), self.weight.data_ptr(), self.eps, self.mult,
-            _lib.ptr(out), ld(out), _lib.ptr(next_weight) if out is not None else None, t, w,
-            _lib.dtype_code(dt), _lib.current_stream())
+            _lib.ptr(b_gate), _lib.ptr(rows), ld(rows), _lib.ptr(row_weights), _lib.ptr(row_ids), int(top),
+            int(experts), _lib.ptr(same), ld(same), self.weight.data_ptr(), self.eps, self.mult,
+            _lib.ptr(table), ld(table), _lib.ptr(table_ids), _lib.ptr(out), ld(out),
+            _lib.ptr(next_weight) if out is not None else None, t, w, _lib.dtype_code(dt), _lib.current_stream())
         _lib.check(rc, "b200_add_normed")
         return out if out is not None else (x if out_dtype == torch.float32 else None)
 
