@@ -549,10 +549,10 @@ def main():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--arch-compare", default=None, metavar="SIZES",
                     help="instead of the headline workload: prefill / decode throughput of the Desirax, "
-                         "Dozetar, Kulesun, Kisilix and Luzosun designs beside the Llama-family stack at equal size ('all' "
+                         "Dozetar, Kulesun, Kisilix, Luzosun and Sapivik designs beside the Llama-family stack at equal size ('all' "
                          "or comma-separated names of model_executor/arch_bench.py SIZES / DOZETAR_SIZES / "
-                         "KULESUN_SIZES / KISILIX_SIZES / LUZOSUN_SIZES, e.g. dz-w1024,ku-w1024,ki-w1024,lu-w1024; a "
-                         "Kulesun size also runs the Desirax stack, a Kisilix size the Dozetar stack, a Luzosun size "
+                         "KULESUN_SIZES / KISILIX_SIZES / LUZOSUN_SIZES / SAPIVIK_SIZES, e.g. dz-w1024,ku-w1024,lu-w1024,sv-w1024; a "
+                         "Kulesun size also runs the Desirax stack, a Kisilix or Sapivik size the Dozetar stack, a Luzosun size "
                          "the Kulesun stack, at equal size); one JSON line per "
                          "model and size")
     args = ap.parse_args()

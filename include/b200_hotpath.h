@@ -908,7 +908,16 @@ int b200_channel_recurrence(const void* q, int64_t ldq, const void* zf, int64_t 
                             int64_t ldv, const float* f_bias, const float* f_lower, float q_scale, int act,
                             float* state, int64_t ld_state, const int64_t* slot, const int* tok_pos,
                             const int* ext_start, const int* ext_len, float* out, int64_t ldo, int batch,
-                            int H, int D, int E, int dtype, void* stream);
+                            int max_len, int H, int D, int E, int dtype, void* stream);
+/* The same for the entries of at least min_len new tokens (longest: max_len), 16 tokens at a time;
+ * b200_channel_recurrence with max_len = min_len > 0 skips exactly those.  D <= 128; work: fp32,
+ * b200_channel_chunks_work(...) values (-1: key size not served), 16-byte aligned.                   */
+int64_t b200_channel_chunks_work(int T, int batch, int H, int D);
+int b200_channel_chunks(const void* q, int64_t ldq, const void* zf, int64_t ldf, const void* v, int64_t ldv,
+                        const float* f_bias, const float* f_lower, float q_scale, int act, float* state,
+                        int64_t ld_state, const int64_t* slot, const int* tok_pos, const int* ext_start,
+                        const int* ext_len, float* out, int64_t ldo, float* work, int T, int batch,
+                        int min_len, int max_len, int H, int D, int E, int dtype, void* stream);
 /* b200_sink_attn with a soft cap (0: none) and an element-wise output gate: out *= sigmoid(gate[t, h, e])
  * (gate [T rows of ld_gate] in the pool's dtype, NULL: none).                                        */
 int b200_sink_attn_gated(const float* q, int64_t ldq, const void* pool, int64_t ld_pool, int k_off,

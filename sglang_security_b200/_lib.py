@@ -312,7 +312,12 @@ _SIGNATURES = {
     "b200_channel_recurrence": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
                                         c_void_p, c_float, c_int, c_void_p, c_int64, c_void_p, c_void_p,
                                         c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int,
-                                        c_int, c_void_p]),
+                                        c_int, c_int, c_void_p]),
+    "b200_channel_chunks_work": (c_int64, [c_int, c_int, c_int, c_int]),
+    "b200_channel_chunks": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                                    c_void_p, c_float, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p,
+                                    c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                    c_int, c_int, c_int, c_void_p]),
     "b200_sink_attn_gated": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_int64,
                                      c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int,
                                      c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,

@@ -20,6 +20,7 @@
 //               (M128 N=D K16 x 4, V consumed as an MN-major B operand); owns the TMEM allocation.
 //   warps 5-7 : gather loaders (cp.async double buffer, slot ids from req_to_token).
 // Two CTAs are co-resident per SM so one CTA's softmax overlaps the other's MMAs.
+#include <cmath>
 #include <cstdlib>
 #include <type_traits>
 
@@ -61,6 +62,8 @@ struct ExtendParams {
   int64_t gate_stride;           // sigmoid(gate[row, head * D + d])
   float score_bound;             // > 0: no capped score exceeds it (unit-norm queries and keys), so it is the
                                  // reference of every exponent instead of the cap; 0: the cap itself
+  float cap_poly[5];             // FAST == 2: cap * log2(e) * tanh(x) / x = sum_i cap_poly[i] x^(2i) on the
+                                 // range the scores can take
 };
 
 constexpr int kExtThreads = 256;
@@ -108,7 +111,11 @@ __device__ __forceinline__ float fmax3(float a, float b, float c) {
 // packed FFMA2 per two elements (exp2(s * scale - m)), and the row sum accumulates with FFMA2.
 // Same values up to fp32 rounding of the fused multiply-add.  Not used with logit capping or a
 // non-positive scale (dispatch falls back to the FAST = false instance, unchanged from round 1).
-template <typename T, int D, bool FAST = false, int NV = 1>
+// FAST == 2: capped scores whose bound keeps |x| = |raw * scale / cap| below kCapPolyMax: tanh is a polynomial
+// there (fitted by the host to the range), so a score costs one exponential, as without a cap, and packed
+// multiply-adds instead of an exponential and a division; the bound is the reference of every exponent.
+constexpr float kCapPolyMax = 0.8f;
+template <typename T, int D, int FAST = 0, int NV = 1>
 __global__ void __launch_bounds__(kExtThreads, 2)
 attn_extend_kernel(const ExtendParams p) {
   using C = ExtendCfg<D, NV>;
@@ -305,7 +312,7 @@ attn_extend_kernel(const ExtendParams p) {
     // the reference of every exponent: exp2(s - r) = exp2((cap - r) - 2 cap / (e^(2x) + 1)) with
     // x = raw * scale / cap.  No running maximum, no rescaling of O, one pass over the tile (the host takes
     // this form for references whose e^(-2 r) stays a normal number)
-    const bool lean_cap = FAST && capped;
+    const bool lean_cap = FAST == 2 || (FAST && capped);
     const float cap_k1 = p.qk_scale * inv_cap * 2.8853900817779268f, cap_k2 = -2.0f * cap_log2;
     const float ref_log2 = p.score_bound > 0.f ? fminf(p.score_bound * 1.4426950408889634f, cap_log2) : cap_log2;
     const float cap_k0 = cap_log2 - ref_log2;
@@ -397,13 +404,34 @@ attn_extend_kernel(const ExtendParams p) {
       uint32_t packed[2][16];
       const float2 sc2 = make_float2(p.qk_scale, p.qk_scale), nm2 = make_float2(-m_use, -m_use);
       const float2 one2 = make_float2(1.f, 1.f);
+      const float2 ref2 = make_float2(-ref_log2, -ref_log2);
+      const float2 cap_x2 = make_float2(p.qk_scale * inv_cap, p.qk_scale * inv_cap);
+      float2 poly2[5];
+#pragma unroll
+      for (int i = 0; i < 5; ++i) poly2[i] = make_float2(p.cap_poly[i], p.cap_poly[i]);
       float2 lsum = make_float2(0.f, 0.f);
 #pragma unroll
       for (int h = 0; h < 2; ++h)
 #pragma unroll
         for (int c = 0; c < 16; ++c) {
           float p0, p1;
-          if (lean_cap) {
+          if constexpr (FAST == 2) {
+            const float2 x = fmul2(make_float2(__uint_as_float(v[h][2 * c]), __uint_as_float(v[h][2 * c + 1])), cap_x2);
+            const float2 y = fmul2(x, x);
+            float2 q = ffma2(y, poly2[4], poly2[3]);
+            q = ffma2(y, q, poly2[2]);
+            q = ffma2(y, q, poly2[1]);
+            q = ffma2(y, q, poly2[0]);
+            q = ffma2(x, q, ref2);
+            p0 = fast_exp2(q.x);
+            p1 = fast_exp2(q.y);
+            if (edge) {
+              const int kp = k0 + h * 32 + 2 * c;
+              if (kp > limit || (kp < first && kp >= kept)) p0 = 0.f;
+              if (kp + 1 > limit || (kp + 1 < first && kp + 1 >= kept)) p1 = 0.f;
+            }
+            lsum = ffma2(make_float2(p0, p1), one2, lsum);
+          } else if (lean_cap) {
             const float e0 = fast_exp2(__uint_as_float(v[h][2 * c]) * cap_k1);
             const float e1 = fast_exp2(__uint_as_float(v[h][2 * c + 1]) * cap_k1);
             p0 = fast_exp2(__fdividef(cap_k2, e0 + 1.0f) + cap_k0);
@@ -518,7 +546,7 @@ static bool extend_fast_softmax_enabled() {
   return !(e && e[0] == '0');
 }
 
-template <typename T, int D, bool FAST, int NV = 1>
+template <typename T, int D, int FAST, int NV = 1>
 static int launch_extend_inst(const ExtendParams& p, int bs, int max_extend_len, cudaStream_t st) {
   using C = ExtendCfg<D, NV>;
   static_assert(C::SMEM_BYTES <= 227 * 1024, "tiles exceed shared memory");
@@ -539,6 +567,28 @@ static int launch_extend_inst(const ExtendParams& p, int bs, int max_extend_len,
   return 0;
 }
 
+// c[i] of mult * tanh(x) / x = sum_i c[i] x^(2i), i < 5, |x| <= range: interpolation in y = x^2 at the Chebyshev
+// nodes of [0, range^2].  tanh's nearest pole lies at y = -(pi / 2)^2, so for range <= 0.8 the relative error
+// stays below 1e-6, and it falls with the tenth power of the range.
+static void fit_cap_polynomial(double mult, double range, float* c) {
+  constexpr int N = 5;
+  const double r2 = 1.02 * range * range + 1e-12, pi = 3.14159265358979323846;
+  double x[N], dd[N];
+  for (int i = 0; i < N; ++i) {
+    x[i] = 0.5 * r2 * (1.0 + std::cos((2 * i + 1) * pi / (2.0 * N)));
+    const double u = std::sqrt(x[i]);
+    dd[i] = mult * (u > 1e-9 ? std::tanh(u) / u : 1.0);
+  }
+  for (int k = 1; k < N; ++k)                  // divided differences (Newton form)
+    for (int i = N - 1; i >= k; --i) dd[i] = (dd[i] - dd[i - 1]) / (x[i] - x[i - k]);
+  double a[N] = {dd[N - 1], 0.0, 0.0, 0.0, 0.0};
+  for (int k = N - 2; k >= 0; --k) {           // a <- a * (y - x[k]) + dd[k]
+    for (int i = N - 1; i >= 1; --i) a[i] = a[i - 1] - x[k] * a[i];
+    a[0] = dd[k] - x[k] * a[0];
+  }
+  for (int i = 0; i < N; ++i) c[i] = static_cast<float>(a[i]);
+}
+
 template <typename T, int D>
 static int launch_extend(const ExtendParams& p, int n_values, int bs, int max_extend_len, cudaStream_t st) {
   // a cap up to 40 keeps e^(-2 cap) a normal fp32 (and 16-bit) number: the one-pass capped form
@@ -546,10 +596,17 @@ static int launch_extend(const ExtendParams& p, int n_values, int bs, int max_ex
   const bool fast = ref <= 40.f && p.qk_scale > 0.f && extend_fast_softmax_enabled();
   note_variant("attn_extend d=%d fast_softmax=%d values=%d", D, fast ? 1 : 0, n_values);
   if (n_values == 2)
-    return fast ? launch_extend_inst<T, D, true, 2>(p, bs, max_extend_len, st)
-                : launch_extend_inst<T, D, false, 2>(p, bs, max_extend_len, st);
-  return fast ? launch_extend_inst<T, D, true>(p, bs, max_extend_len, st)
-              : launch_extend_inst<T, D, false>(p, bs, max_extend_len, st);
+    return fast ? launch_extend_inst<T, D, 1, 2>(p, bs, max_extend_len, st)
+                : launch_extend_inst<T, D, 0, 2>(p, bs, max_extend_len, st);
+  if (fast && p.logit_cap > 0.f && p.score_bound > 0.f && p.score_bound < p.logit_cap * std::tanh(kCapPolyMax)) {
+    ExtendParams pp = p;
+    fit_cap_polynomial(p.logit_cap * 1.4426950408889634, std::atanh(static_cast<double>(p.score_bound) / p.logit_cap),
+                       pp.cap_poly);
+    note_variant("attn_extend d=%d cap_polynomial", D);
+    return launch_extend_inst<T, D, 2>(pp, bs, max_extend_len, st);
+  }
+  return fast ? launch_extend_inst<T, D, 1>(p, bs, max_extend_len, st)
+              : launch_extend_inst<T, D, 0>(p, bs, max_extend_len, st);
 }
 
 }  // namespace b200

@@ -41,7 +41,7 @@
 //                         Gate mode 1: o is multiplied by silu(z) BEFORE the norm instead.
 #include <cstdlib>
 
-#include "common.cuh"
+#include "f32x2.cuh"
 
 namespace b200 {
 
@@ -54,27 +54,6 @@ __device__ __forceinline__ float rec_act(float z, int act) {
 }
 __device__ __forceinline__ void cp_async8(uint32_t smem_addr, const void* gptr) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 8;\n" ::"r"(smem_addr), "l"(gptr));
-}
-// two fp32 lanes in one 64-bit register: the packed multiply-adds below take and return these, so no
-// instruction is spent on pairing registers
-using f32x2 = unsigned long long;
-__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
-  f32x2 r;
-  asm("mov.b64 %0, {%1, %2};\n" : "=l"(r) : "f"(lo), "f"(hi));
-  return r;
-}
-__device__ __forceinline__ void unpack2(f32x2 v, float& lo, float& hi) {
-  asm("mov.b64 {%0, %1}, %2;\n" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
-  f32x2 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
-  f32x2 d;
-  asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
-  return d;
 }
 __device__ __forceinline__ float log_sigmoid(float z) {
   return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
@@ -92,7 +71,7 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
                          const int* __restrict__ ext_start, const int* __restrict__ ext_len,
                          float* __restrict__ out, int64_t ldo, float* __restrict__ aux, int64_t ld_aux,
                          int H, int D, int E, int P, int CH, int stream_rows,
-                         const float* __restrict__ f_bias, const float* __restrict__ f_lower) {
+                         const float* __restrict__ f_bias, const float* __restrict__ f_lower, int max_len) {
   constexpr bool GATES = FORM == 1;
   extern __shared__ __align__(16) float rec_smem[];
   const int nthreads = blockDim.x, nwarps = nthreads >> 5;
@@ -112,7 +91,7 @@ linear_recurrence_kernel(const T* __restrict__ q, int64_t ldq, const T* __restri
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int p = tid % P, cp = tid / P, e = e0 + 2 * cp;
   const int start = ext_start[b], len = ext_len[b];
-  if (len <= 0) return;
+  if (len <= 0 || (max_len > 0 && len >= max_len)) return;
   const bool fresh = tok_pos[start] == 0;
   const int ncols = E + (GATES ? 1 : 0);      // the gated form's last column is the normaliser (v = 1)
   const int NCP = (ncols + 1) / 2, D4 = (D + 3) / 4;
@@ -374,7 +353,7 @@ static int linear_recurrence_impl(const void* q, int64_t ldq, const void* k, int
                                   float cap, float q_scale, int act, float* state, int64_t ld_state,
                                   const int64_t* slot, const int* tok_pos, const int* ext_start,
                                   const int* ext_len, float* out, int64_t ldo, float* aux, int64_t ld_aux,
-                                  int batch, int H, int D, int E, int dtype, void* stream) {
+                                  int batch, int max_len, int H, int D, int E, int dtype, void* stream) {
   using namespace b200;
   if (batch == 0) return 0;
   B200_REQUIRE(q && k && v && state && slot && tok_pos && ext_start && ext_len && out,
@@ -434,7 +413,7 @@ static int linear_recurrence_impl(const void* q, int64_t ldq, const void* k, int
     launch_kernel(kern, grid, dim3(nthreads), smem, st, 1, 0, static_cast<const TT*>(q), ldq,        \
                   static_cast<const TT*>(k), ldk, static_cast<const TT*>(v), ldv, gates, ldg, decay, \
                   cap, q_scale, act, state, ld_state, slot, tok_pos, ext_start, ext_len, out, ldo,   \
-                  aux, ld_aux, H, D, E, P, CH, stream_rows ? 1 : 0, f_bias, f_lower);                \
+                  aux, ld_aux, H, D, E, P, CH, stream_rows ? 1 : 0, f_bias, f_lower, max_len);       \
   } while (0)
 #define BY_G(TT)                  \
   do {                            \
@@ -463,19 +442,21 @@ extern "C" int b200_linear_recurrence(const void* q, int64_t ldq, const void* k,
                                       int H, int D, int E, int dtype, void* stream) {
   return linear_recurrence_impl(q, ldq, k, ldk, v, ldv, gates, ldg, decay, nullptr, nullptr, gates ? 1 : 0, cap,
                                 q_scale, act, state, ld_state, slot, tok_pos, ext_start, ext_len, out, ldo, aux,
-                                ld_aux, batch, H, D, E, dtype, stream);
+                                ld_aux, batch, 0, H, D, E, dtype, stream);
 }
 
 // The channel form: zf [T, H * D] are the forget gate's pre-activations, f_bias / f_lower fp32 [H * D] its
-// bias and lower bound (NULL: zero), act 1: silu on the queries.
+// bias and lower bound (NULL: zero), act 1: silu on the queries.  max_len > 0: entries of at least max_len new
+// tokens are skipped (b200_channel_chunks walks those).
 extern "C" int b200_channel_recurrence(const void* q, int64_t ldq, const void* zf, int64_t ldf, const void* v,
                                        int64_t ldv, const float* f_bias, const float* f_lower, float q_scale,
                                        int act, float* state, int64_t ld_state, const int64_t* slot,
                                        const int* tok_pos, const int* ext_start, const int* ext_len, float* out,
-                                       int64_t ldo, int batch, int H, int D, int E, int dtype, void* stream) {
+                                       int64_t ldo, int batch, int max_len, int H, int D, int E, int dtype,
+                                       void* stream) {
   return linear_recurrence_impl(q, ldq, zf, ldf, v, ldv, nullptr, 0, nullptr, f_bias, f_lower, 2, 0.f, q_scale, act,
                                 state, ld_state, slot, tok_pos, ext_start, ext_len, out, ldo, nullptr, 0, batch,
-                                H, D, E, dtype, stream);
+                                max_len, H, D, E, dtype, stream);
 }
 
 // aux (optional): fp32 [T, 2 H] = (n . q, m) of the gated recurrence; o is divided by

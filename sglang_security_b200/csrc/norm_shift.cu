@@ -18,7 +18,8 @@
 //                          rows[t * top + k] : same[t]) — a per-token gate on b, weighted expert rows, identity
 //                          experts that return their input —, then x as above, then x += table[id_t] (a row of
 //                          an embedding table, ahead of the next pass of a loop), then the copy / pre-norm.  16-byte
-//                          loads, y and x stay in registers between the two norms.
+//                          loads, y and x stay in registers between the two norms (wide or unaligned rows: in shared
+//                          memory).
 //   softcap_rows         : out = cap * tanh(z / cap) in fp32
 //   scaled_add_layernorm : for designs whose norm sits AFTER the residual sum: y = alpha * x + a + b +
 //                          sum_k wts[t, k] * rows[t * top + k] (terms optional) in fp32, then
@@ -191,17 +192,53 @@ __device__ __forceinline__ float block_sum_any(float v, float* red) {
   return t;
 }
 
-// acc[i] += s * p[i] for V consecutive values (V = 1, or one 16-byte load)
+// acc[i] += s * p[i] for the V consecutive values of one 16-byte load
 template <typename TA, int V>
 __device__ __forceinline__ void axpy_load(float (&acc)[V], float s, const TA* p) {
-  if constexpr (V == 1) {
-    acc[0] = fmaf(s, to_float<TA>(*p), acc[0]);
-  } else {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
-    const TA* e = reinterpret_cast<const TA*>(&u);
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const TA* e = reinterpret_cast<const TA*>(&u);
 #pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = fmaf(s, to_float<TA>(e[i]), acc[i]);
+  for (int i = 0; i < V; ++i) acc[i] = fmaf(s, to_float<TA>(e[i]), acc[i]);
+}
+
+// Any width and alignment: the summed row, then the new residual row, stay in shared memory.
+template <typename TA>
+__global__ void __launch_bounds__(kRowThreads)
+add_normed_mix_any_kernel(const AddNormedMix p) {
+  extern __shared__ float mix_row[];
+  __shared__ float red[kRowThreads / 32];
+  const int64_t t = blockIdx.x;
+  const int W = p.W;
+  const float gb = p.b ? (p.gb ? p.gb[t] : 1.f) * p.sb : 0.f;
+  float s = 0.f;
+  for (int d = threadIdx.x; d < W; d += kRowThreads) {
+    float v = 0.f;
+    if (p.a) v = fmaf(p.sa, to_float<TA>(static_cast<const TA*>(p.a)[t * p.lda + d]), v);
+    if (p.b) v = fmaf(gb, to_float<TA>(static_cast<const TA*>(p.b)[t * p.ldb + d]), v);
+    if (p.rows)
+      for (int k = 0; k < p.top; ++k) {
+        const bool own = p.ids && p.ids[t * p.top + k] >= p.n_experts;
+        const TA* src = own ? static_cast<const TA*>(p.same) + t * p.ld_same
+                            : static_cast<const TA*>(p.rows) + (t * p.top + k) * p.ld_rows;
+        v = fmaf(p.wts ? p.wts[t * p.top + k] : 1.f, to_float<TA>(src[d]), v);
+      }
+    mix_row[d] = v;
+    s = fmaf(v, v, s);
   }
+  const float r = p.mult / sqrtf(block_sum(s, red) / static_cast<float>(W) + p.eps);
+  const TA* extra = p.table ? static_cast<const TA*>(p.table) + p.table_ids[t] * p.ld_table : nullptr;
+  float s2 = 0.f;
+  for (int d = threadIdx.x; d < W; d += kRowThreads) {
+    float nx = fmaf(mix_row[d] * r, p.w ? p.w[d] : 1.f, p.x[t * p.ldx + d]);
+    if (extra) nx += to_float<TA>(extra[d]);
+    p.x[t * p.ldx + d] = nx;
+    mix_row[d] = nx;
+    s2 = fmaf(nx, nx, s2);
+  }
+  if (!p.out_h) return;
+  const float r2 = p.w_next ? 1.0f / sqrtf(block_sum(s2, red) / static_cast<float>(W) + p.eps) : 1.f;
+  for (int d = threadIdx.x; d < W; d += kRowThreads)
+    static_cast<TA*>(p.out_h)[t * p.ldh + d] = from_float<TA>(mix_row[d] * r2 * (p.w_next ? p.w_next[d] : 1.f));
 }
 
 // A thread owns NC chunks of V consecutive coordinates of one token's row.
@@ -222,7 +259,7 @@ add_normed_mix_kernel(const AddNormedMix p) {
     if (d < W) {
       if (p.a) axpy_load<TA, V>(y[c], p.sa, static_cast<const TA*>(p.a) + t * p.lda + d);
       if (p.b) axpy_load<TA, V>(y[c], gb, static_cast<const TA*>(p.b) + t * p.ldb + d);
-      if (p.rows || p.ids) {
+      if (p.rows) {
 #pragma unroll 4
         for (int k = 0; k < p.top; ++k) {
           const float wk = p.wts ? p.wts[t * p.top + k] : 1.f;
@@ -245,9 +282,6 @@ add_normed_mix_kernel(const AddNormedMix p) {
     if (d < W) {
       float* xr = p.x + t * p.ldx + d;
       float nx[V];
-      if constexpr (V == 1) {
-        nx[0] = fmaf(y[c][0] * r, p.w ? p.w[d] : 1.f, xr[0]);
-      } else {
 #pragma unroll
         for (int i = 0; i < V; i += 4) {
           const float4 xv = *reinterpret_cast<const float4*>(xr + i);
@@ -257,15 +291,10 @@ add_normed_mix_kernel(const AddNormedMix p) {
           nx[i + 2] = fmaf(y[c][i + 2] * r, wv.z, xv.z);
           nx[i + 3] = fmaf(y[c][i + 3] * r, wv.w, xv.w);
         }
-      }
       if (extra) axpy_load<TA, V>(nx, 1.f, extra + d);
-      if constexpr (V == 1) {
-        xr[0] = nx[0];
-      } else {
 #pragma unroll
-        for (int i = 0; i < V; i += 4)
-          *reinterpret_cast<float4*>(xr + i) = make_float4(nx[i], nx[i + 1], nx[i + 2], nx[i + 3]);
-      }
+      for (int i = 0; i < V; i += 4)
+        *reinterpret_cast<float4*>(xr + i) = make_float4(nx[i], nx[i + 1], nx[i + 2], nx[i + 3]);
 #pragma unroll
       for (int i = 0; i < V; ++i) {
         s2 = fmaf(nx[i], nx[i], s2);
@@ -284,9 +313,6 @@ add_normed_mix_kernel(const AddNormedMix p) {
     const int d = (c * blockDim.x + threadIdx.x) * V;
     if (d >= W) continue;
     TA* dst = static_cast<TA*>(p.out_h) + t * p.ldh + d;
-    if constexpr (V == 1) {
-      dst[0] = from_float<TA>(y[c][0] * r2 * (p.w_next ? p.w_next[d] : 1.f));
-    } else {
       uint4 u;
       TA* e = reinterpret_cast<TA*>(&u);
 #pragma unroll
@@ -298,7 +324,6 @@ add_normed_mix_kernel(const AddNormedMix p) {
         e[i + 3] = from_float<TA>(y[c][i + 3] * r2 * wv.w);
       }
       *reinterpret_cast<uint4*>(dst) = u;
-    }
   }
 }
 
@@ -473,22 +498,24 @@ extern "C" int b200_add_normed_mix(float* x, int64_t ldx, const void* a, int64_t
   const bool vec = W % v == 0 && aligned16(x) && ldx % 4 == 0 && fits(a, lda) && fits(b, ldb) && fits(rows, ld_rows) &&
                    fits(same, ld_same) && fits(table, ld_table) && fits(out_h, ldh) && aligned16(w) && aligned16(w_next) &&
                    W <= v * kRowThreads * 4;
-  const int chunks = vec ? W / v : W;
-  int nc = 1;
-  while (nc * kRowThreads < chunks) nc <<= 1;
-  B200_REQUIRE(nc <= 32, "b200_add_normed_mix: width %d too large for unaligned rows", W);
-  int nt = min(kRowThreads, ceil_div(ceil_div(chunks, nc), 32) * 32);
+  const int nc = W <= v * kRowThreads ? 1 : (W <= v * kRowThreads * 2 ? 2 : 4);
+  const int nt = ceil_div(ceil_div(W / v, nc), 32) * 32;
+  const size_t smem = sizeof(float) * static_cast<size_t>(W);
+  B200_REQUIRE(vec || smem <= 200 * 1024, "b200_add_normed_mix: width %d too large", W);
 #define LAUNCH(TA, V, NC) launch_kernel(add_normed_mix_kernel<TA, V, NC>, dim3(T), dim3(nt), 0, st, 1, 0, p)
 #define BY_NC(TA, V)                                                                                 \
   do {                                                                                               \
-    if (vec) {                                                                                       \
-      if (nc == 1) LAUNCH(TA, V, 1);                                                                 \
-      else if (nc == 2) LAUNCH(TA, V, 2);                                                            \
-      else LAUNCH(TA, V, 4);                                                                         \
-    } else if (nc <= 4) {                                                                            \
-      LAUNCH(TA, 1, 4);                                                                              \
+    if (!vec) {                                                                                      \
+      if (smem > 48 * 1024)                                                                          \
+        B200_CUDA_OK(cudaFuncSetAttribute(add_normed_mix_any_kernel<TA>,                             \
+                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));  \
+      launch_kernel(add_normed_mix_any_kernel<TA>, dim3(T), dim3(kRowThreads), smem, st, 1, 0, p);   \
+    } else if (nc == 1) {                                                                            \
+      LAUNCH(TA, V, 1);                                                                              \
+    } else if (nc == 2) {                                                                            \
+      LAUNCH(TA, V, 2);                                                                              \
     } else {                                                                                         \
-      LAUNCH(TA, 1, 32);                                                                             \
+      LAUNCH(TA, V, 4);                                                                              \
     }                                                                                                \
   } while (0)
   if (dtype == B200_BF16) BY_NC(__nv_bfloat16, 8);

@@ -181,6 +181,93 @@ qk_norm_rope_write_kernel(const T* __restrict__ q, int64_t ldq, const T* __restr
   }
 }
 
+// The same for 16-bit rows, head sizes 64 / 128 / 256 and norms per head (or none): four warps per token, a warp
+// takes every fourth head, a lane VN = D / 32 consecutive coordinates (whole rotation pairs), so a head is one
+// vector load, one shuffle tree and one vector store, and the sines and cosines a lane needs are the same for
+// all heads.  Values that are the projected keys (v == k) are written from the registers that hold them.
+constexpr int kHeadPrepWarps = 4;
+
+template <typename T, int VN>
+__global__ void __launch_bounds__(kHeadPrepWarps * 32)
+qk_head_rope_write_kernel(const T* __restrict__ q, int64_t ldq, const T* __restrict__ k, int64_t ldk,
+                          const T* __restrict__ v, int64_t ldv, const float* __restrict__ qw,
+                          const float* __restrict__ kw, int q_norm, int k_norm, float eps,
+                          const float* __restrict__ freq_hi, const float* __restrict__ freq_lo, int rot_dims,
+                          const int* __restrict__ tok_pos, const int64_t* __restrict__ loc,
+                          T* __restrict__ pool, int64_t ld_pool, int k_off, int v_off,
+                          float* __restrict__ q_out, int64_t ldqo, T* __restrict__ q_out16, int64_t ldqo16,
+                          int H, int G, int E, float temp_coef, int temp_every) {
+  constexpr int D = 32 * VN;
+  using Vec = typename std::conditional<VN == 2, uint32_t, typename std::conditional<VN == 4, uint2, uint4>::type>::type;
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, d0 = lane * VN;
+  const int p = tok_pos[t];
+  const bool tied = v == k && E == D;
+  float cs[VN / 2], sn[VN / 2];
+#pragma unroll
+  for (int i = 0; i < VN / 2; ++i) {
+    cs[i] = 1.f;
+    sn[i] = 0.f;
+    if (d0 + 2 * i < rot_dims) {
+      const int f = d0 / 2 + i;
+      const float hi = freq_hi[f], lo = freq_lo ? freq_lo[f] : 0.f, pos = static_cast<float>(p), a = pos * hi;
+      const float err = fmaf(pos, hi, -a) + pos * lo;     // what the rounded product dropped
+      float s, c;
+      sincosf(a, &s, &c);
+      cs[i] = c - err * s;
+      sn[i] = s + err * c;
+    }
+  }
+  const float temp = temp_every > 0 ? 1.0f + temp_coef * logf(static_cast<float>((p + 1) / temp_every) + 1.0f) : 1.0f;
+  T* prow = pool + loc[t] * ld_pool;
+#pragma unroll 2
+  for (int hd = warp; hd < H + G; hd += kHeadPrepWarps) {
+    const bool is_q = hd < H;
+    const int g = hd - H;
+    const T* src = is_q ? q + t * ldq + hd * D : k + t * ldk + g * D;
+    const Vec raw = *reinterpret_cast<const Vec*>(src + d0);
+    float x[VN];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VN; ++i) {
+      x[i] = to_float<T>(reinterpret_cast<const T*>(&raw)[i]);
+      ss = fmaf(x[i], x[i], ss);
+    }
+    if (is_q ? q_norm : k_norm) {
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = 1.0f / sqrtf(ss / static_cast<float>(D) + eps);
+      const float* w = is_q ? (qw ? qw + hd * D + d0 : nullptr) : (kw ? kw + g * D + d0 : nullptr);
+#pragma unroll
+      for (int i = 0; i < VN; ++i) x[i] *= w ? inv * w[i] : inv;
+    }
+#pragma unroll
+    for (int i = 0; i < VN / 2; ++i) {
+      const float a = x[2 * i], b = x[2 * i + 1];
+      x[2 * i] = fmaf(a, cs[i], -b * sn[i]);
+      x[2 * i + 1] = fmaf(b, cs[i], a * sn[i]);
+    }
+    Vec packed;
+#pragma unroll
+    for (int i = 0; i < VN; ++i) {
+      if (is_q) x[i] *= temp;
+      reinterpret_cast<T*>(&packed)[i] = from_float<T>(x[i]);
+    }
+    if (is_q) {
+      if (q_out16) *reinterpret_cast<Vec*>(q_out16 + t * ldqo16 + hd * D + d0) = packed;
+      if (q_out) {
+        float* dst = q_out + t * ldqo + hd * D + d0;
+#pragma unroll
+        for (int i = 0; i < VN; i += 2) *reinterpret_cast<float2*>(dst + i) = make_float2(x[i], x[i + 1]);
+      }
+    } else {
+      *reinterpret_cast<Vec*>(prow + k_off + g * D + d0) = packed;
+      if (tied) *reinterpret_cast<Vec*>(prow + v_off + g * D + d0) = raw;
+    }
+  }
+  if (!tied)
+    for (int i = threadIdx.x; i < G * E; i += kHeadPrepWarps * 32) prow[v_off + i] = v[t * ldv + i];
+}
+
 constexpr int kSinkMaxWarps = 16;  // warps per CTA: 4 to 16, by the longest key list (host)
 constexpr int kSinkMaxCols = 8;    // value size <= 256
 constexpr int kSinkHeads = 4;      // query heads of a key/value head scored per pass over its keys
@@ -432,6 +519,34 @@ extern "C" int b200_qkv_prep_write(const void* q, int64_t ldq, const void* k, in
   B200_REQUIRE(smem <= 48 * 1024, "b200_qkv_prep_write: too many norm groups");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   ScopedKernelTimer timer("qk_norm_rope_write", st);
+  const int vn = D / 32;
+  auto rows_of = [&](const void* ptr, int64_t ld) {       // rows that every lane's vector access fits
+    return !ptr || (reinterpret_cast<uintptr_t>(ptr) % (2 * vn) == 0 && ld % vn == 0);
+  };
+  if ((dtype == B200_BF16 || dtype == B200_F16) && (D == 64 || D == 128 || D == 256) &&
+      (q_group == 0 || q_group == D) && (k_group == 0 || k_group == D) && !v_norm && !first_pool &&
+      rows_of(q, ldq) && rows_of(k, ldk) && rows_of(pool, ld_pool) && rows_of(q_out16, ldqo16) &&
+      (!q_out || (reinterpret_cast<uintptr_t>(q_out) % 8 == 0 && ldqo % 2 == 0)) && k_off % vn == 0 &&
+      (v != k || v_off % vn == 0)) {
+#define LAUNCH_H(TT, VN)                                                                             \
+  launch_kernel(qk_head_rope_write_kernel<TT, VN>, dim3(T), dim3(kHeadPrepWarps * 32), 0, st, 1, 0,  \
+                static_cast<const TT*>(q), ldq, static_cast<const TT*>(k), ldk,                      \
+                static_cast<const TT*>(v), ldv, qw, kw, q_group, k_group, eps, freq_hi, freq_lo,     \
+                rot_dims, tok_pos, loc, static_cast<TT*>(pool), ld_pool, k_off, v_off, q_out, ldqo,  \
+                static_cast<TT*>(q_out16), ldqo16, H, G, E, temp_coef, temp_every)
+#define BY_VN(TT)                \
+  do {                           \
+    if (vn == 2) LAUNCH_H(TT, 2); \
+    else if (vn == 4) LAUNCH_H(TT, 4); \
+    else LAUNCH_H(TT, 8);        \
+  } while (0)
+    if (dtype == B200_BF16) BY_VN(__nv_bfloat16);
+    else BY_VN(__half);
+#undef BY_VN
+#undef LAUNCH_H
+    B200_CHECK_LAUNCH("qk_head_rope_write_kernel");
+    return 0;
+  }
 #define LAUNCH(TT)                                                                                   \
   launch_kernel(qk_norm_rope_write_kernel<TT, TT>, dim3(T), dim3(kPrepThreads), smem, st, 1, 0,      \
                 static_cast<const TT*>(q), ldq, static_cast<const TT*>(k), ldk,                      \

@@ -92,9 +92,11 @@ def gated_group_rmsnorm(o: torch.Tensor, weight: Optional[torch.Tensor], z: Opti
 
 def channel_recurrence(q: torch.Tensor, zf: torch.Tensor, v: torch.Tensor, bias: Optional[torch.Tensor],
                        lower: Optional[torch.Tensor], heads: int, dim: int, vdim: int, state: torch.Tensor,
-                       fb, q_scale: float = 1.0, silu: bool = True) -> torch.Tensor:
+                       fb, q_scale: float = 1.0, silu: bool = True, chunk_min: int = 32) -> torch.Tensor:
     """q, zf [T, heads * dim] (zf: the forget gates' pre-activations), v [T, heads * vdim], row-strided views
-    of one dtype; bias, lower fp32 [heads * dim] -> fp32 [T, heads * vdim].  silu applies to q."""
+    of one dtype; bias, lower fp32 [heads * dim] -> fp32 [T, heads * vdim].  silu applies to q.  Portions of at
+    least `chunk_min` tokens (0: none) are walked 16 tokens at a time (csrc/channel_chunks.cu, dim <= 128), the
+    others token by token; both leave the same state."""
     if not q.is_cuda:
         raise _lib.B200Error("channel_recurrence: tensors must live on a CUDA device (no CPU path)")
     for t in (q, zf, v):
@@ -103,13 +105,24 @@ def channel_recurrence(q: torch.Tensor, zf: torch.Tensor, v: torch.Tensor, bias:
     for t in (bias, lower):
         if t is not None and (t.dtype != torch.float32 or t.numel() != heads * dim or not t.is_contiguous()):
             raise _lib.B200Error("channel_recurrence: bias and lower bound are fp32 [heads * dim]")
-    out = torch.empty((q.shape[0], heads * vdim), dtype=torch.float32, device=q.device)
-    rc = _lib.load().b200_channel_recurrence(
-        q.data_ptr(), q.stride(0), zf.data_ptr(), zf.stride(0), v.data_ptr(), v.stride(0), _lib.ptr(bias),
-        _lib.ptr(lower), float(q_scale), 1 if silu else 0, state.data_ptr(), state.stride(0),
-        fb.req_pool_indices.data_ptr(), fb.tok_pos.data_ptr(), fb.ext_start.data_ptr(), fb.ext_len.data_ptr(),
-        out.data_ptr(), out.stride(0), int(fb.batch_size), heads, dim, vdim, _lib.dtype_code(q.dtype),
-        _lib.current_stream())
+    T, lib, lens = q.shape[0], _lib.load(), fb.extend_seq_lens_cpu
+    out = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
+    args = (q.data_ptr(), q.stride(0), zf.data_ptr(), zf.stride(0), v.data_ptr(), v.stride(0), _lib.ptr(bias),
+            _lib.ptr(lower), float(q_scale), 1 if silu else 0, state.data_ptr(), state.stride(0),
+            fb.req_pool_indices.data_ptr(), fb.tok_pos.data_ptr(), fb.ext_start.data_ptr(), fb.ext_len.data_ptr(),
+            out.data_ptr(), out.stride(0))
+    tail = (heads, dim, vdim, _lib.dtype_code(q.dtype), _lib.current_stream())
+    longest = max(lens) if chunk_min > 0 and dim <= 128 else 0
+    if longest >= max(chunk_min, 1):
+        work = torch.empty(int(lib.b200_channel_chunks_work(T, int(fb.batch_size), heads, dim)), dtype=torch.float32,
+                           device=q.device)
+        rc = lib.b200_channel_chunks(*args, work.data_ptr(), T, int(fb.batch_size), chunk_min, longest, *tail)
+        _lib.check(rc, "b200_channel_chunks")
+        if min(lens) >= chunk_min:
+            return out
+    else:
+        chunk_min = 0
+    rc = lib.b200_channel_recurrence(*args, int(fb.batch_size), chunk_min, *tail)
     _lib.check(rc, "b200_channel_recurrence")
     return out
 

@@ -1,11 +1,13 @@
-"""Prefill and decode throughput of the Desirax, Dozetar, Kulesun, Kisilix and Luzosun designs at layer sizes that
+"""Prefill and decode throughput of the Desirax, Dozetar, Kulesun, Kisilix, Luzosun and Sapivik designs at layer sizes that
 resemble a real model's, beside the Llama-family decoder stack of this package at equal width / heads / head size /
 layer count and equal active feed-forward size (random weights, bf16).  Driven by
 `bench.py --arch-compare` (sizes named "dz-..." are Dozetar's, "ku-..." Kulesun's; a Kulesun size also
 runs the Desirax stack, its closest relative, at equal width, heads, latent sizes, layers and feed-forward;
 "ki-..." are Kisilix's, which also run the Dozetar stack — recurrent memories of the same shape, windowed
 attention with the same heads, experts of the same size; "lu-..." are Luzosun's, which also run the Kulesun
-stack — 32-bit residual, dense feed-forward of the same size, attention with the same heads).
+stack — 32-bit residual, dense feed-forward of the same size, attention with the same heads; "sv-..." are
+Sapivik's, which also run the Dozetar stack — decayed memories of the same shape, attention with the same heads
+and no window, experts of the same size).
 
 Timing: CUDA events on the launching stream around whole engine steps, after warm-up steps; every step
 touches more weight and cache bytes than L2 holds at the larger size.  Per-kernel times come from the
@@ -63,6 +65,16 @@ LUZOSUN_SIZES = {
     "lu-w1024": dict(KULESUN_SIZES["ku-w1024"], chunk=8192, conv=4, taps=4),
     "lu-w2048": dict(KULESUN_SIZES["ku-w2048"], kv_heads=4, chunk=8192, conv=4, taps=4),
     "lu-w2048-c512": dict(KULESUN_SIZES["ku-w2048"], kv_heads=4, chunk=512, conv=4, taps=4),
+}
+# Sapivik: channel-gated memory and tied attention alternate, experts (some of them identity experts) with a
+# gated shared expert in every layer; "-dense": clamped gated feed-forwards of the Llama-like stack's size.  The
+# memories have the shape of Dozetar's in the same row, the attention its heads without a window.
+SAPIVIK_SIZES = {
+    "sv-w1024": dict(DOZETAR_SIZES["dz-w1024"], window=1 << 20, keep_first=0, r_dim=64, identity=2, shared=1024, dense=0),
+    "sv-w2048": dict(DOZETAR_SIZES["dz-w2048"], window=1 << 20, keep_first=0, r_dim=128, identity=4, shared=1024,
+                     dense=0),
+    "sv-w2048-dense": dict(DOZETAR_SIZES["dz-w2048"], window=1 << 20, keep_first=0, r_dim=128, identity=4, shared=1024,
+                           ff=8192, dense=8192),
 }
 WORK = dict(prefill_reqs=4, prefill_len=2048, decode_bs=32, decode_ctx=2048)
 
@@ -628,6 +640,110 @@ def bench_luzosun(name, s, steps, warmup, device="cuda"):
     return row
 
 
+def _sapivik_cfg(s):
+    mem = {"type": "hgrn2", "mixer": {"heads": s["r_heads"], "dim": s["r_dim"], "vdim": s["r_vdim"]}}
+    att = {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"],
+                                          "scale": s["dim"] ** -0.5, "softcap": 50.0,
+                                          "rot": {"base": 1e6, "dims": s["rot"]}}}
+    f = {"kind": "moe", "router": {"experts": s["experts"], "identity": s["identity"], "top": s["top"], "scale": 2.0},
+         "expert": {"ff": s["expert_ff"]}, "shared": {"ff": s["shared"]}}
+    if s["dense"]:
+        f = {"kind": "dense", "ff": s["dense"], "limit": 7.0}
+    return {"architecture": "Sapivik", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "residual_mult": 0.5, "layers": [dict(mem if i % 2 == 0 else att, mlp=f) for i in range(s["layers"])]}
+
+
+def bench_sapivik(name, s, steps, warmup, device="cuda"):
+    from ..configs.sapivik import sapivik_config
+    from ..managers.schedule_batch import Req, StepItem
+    from ..managers.scheduler import Scheduler
+    from ..models.registry import resolve_model_cls
+    from .model_runner import ModelRunner
+
+    cfg = sapivik_config(_sapivik_cfg(s))
+    torch.manual_seed(0)
+    with torch.device(device):
+        model = resolve_model_cls("Sapivik")(cfg, params_dtype=torch.bfloat16)
+    for n_, p in model.named_parameters():
+        if n_.endswith("norm_weight") or ("norm" in n_ and n_.endswith(".weight")):
+            p.data.fill_(1.0)
+        elif n_.endswith("f_bias"):
+            p.data.fill_(2.0)
+        elif n_.endswith("f_lower"):
+            p.data.fill_(0.5)
+        elif n_.endswith("correction"):
+            p.data.zero_()
+        else:
+            p.data.normal_(0, 0.02)
+    W = WORK
+    bs = max(W["prefill_reqs"], W["decode_bs"])
+    tokens = W["decode_bs"] * (W["decode_ctx"] + 64) + W["prefill_reqs"] * W["prefill_len"]
+    runner = ModelRunner(None, torch.bfloat16, max_total_tokens=tokens, max_running_requests=bs + 1,
+                         context_length=max(W["prefill_len"], W["decode_ctx"] + 64), device=device,
+                         model=model.eval(), model_config=SimpleNamespace(architecture="Sapivik", hf_config=cfg))
+    sched = Scheduler(runner)
+    g = torch.Generator().manual_seed(1)
+    rnd = lambda n: torch.randint(0, s["vocab"], (n,), generator=g).tolist()
+
+    def prefill():
+        reqs = [Req(rid=f"p{i}", input_ids=rnd(W["prefill_len"])) for i in range(W["prefill_reqs"])]
+        for r in reqs:
+            assert runner.admit(r)
+        sched.run_step([StepItem(r, r.input_ids, want=[len(r.input_ids) - 1]) for r in reqs])
+        for r in reqs:
+            runner.release(r)
+
+    names = ["channel_recurrence", "channel_prepare", "channel_chunks", "channel_scan", "gated_group_rmsnorm",
+             "attn_extend", "attn_decode_split", "attn_merge",
+             "sink_attn", "qk_norm_rope_write", "moe_grouped_gemm", "moe_route", "moe_align", "add_normed",
+             "act_and_mul", "act_and_mul_clamped", "dense_gemm"]
+    row = {"arch": "sapivik", "size": name}
+    ms = _timed(prefill, steps, warmup)
+    ntok = W["prefill_reqs"] * W["prefill_len"]
+    row["prefill_ms"], row["prefill_tokens_per_s"] = round(ms, 3), round(ntok / ms * 1e3)
+    row["prefill_kernels"] = _kernel_times(prefill, names)
+    reqs = [Req(rid=f"d{i}", input_ids=rnd(W["decode_ctx"])) for i in range(W["decode_bs"])]
+    for r in reqs:
+        assert runner.admit(r)
+    for i in range(0, len(reqs), 4):
+        sched.run_step([StepItem(r, r.input_ids) for r in reqs[i:i + 4]])
+    state = {"n": 0}
+
+    def decode():
+        state["n"] += 1
+        assert state["n"] < 60
+        sched.run_step([StepItem(r, [7], want=[0]) for r in reqs])
+
+    ms = _timed(decode, steps, warmup)
+    row["decode_ms"], row["decode_tokens_per_s"] = round(ms, 3), round(W["decode_bs"] / ms * 1e3)
+    row["decode_kernels"] = _kernel_times(decode, names)
+
+    def mixed():
+        state["n"] += 1
+        assert state["n"] < 60
+        new = Req(rid=f"m{state['n']}", input_ids=rnd(512))
+        assert runner.admit(new)
+        sched.run_step([StepItem(r, [7], want=[0]) for r in reqs] + [StepItem(new, new.input_ids, want=[511])])
+        runner.release(new)
+
+    row["mixed_ms"] = round(_timed(mixed, min(steps, 8), 3), 3)
+    # algorithmic work of one launch (all tokens, one layer)
+    L, U, H, G, D = W["prefill_len"], W["prefill_reqs"], s["heads"], s["kv_heads"], s["dim"]
+    n = U * L
+    row["attn_prefill_flops"] = 4 * U * (L * (L + 1) // 2) * H * D
+    row["attn_decode_bytes"] = W["decode_bs"] * (W["decode_ctx"] + 1) * G * 2 * D * 2
+    # three fp32 multiply-adds per memory element and token (difference, write, read-out)
+    row["memory_prefill_fma"] = 3 * n * s["r_heads"] * s["r_dim"] * s["r_vdim"]
+    row["memory_decode_bytes"] = 2 * 4 * W["decode_bs"] * s["r_heads"] * s["r_dim"] * s["r_vdim"]
+    row["expert_prefill_flops"] = 2 * 3 * n * s["top"] * s["expert_ff"] * s["width"] * s["experts"] // (
+        s["experts"] + s["identity"])                              # what the identity experts take needs none
+    row["add_normed_bytes"] = n * s["width"] * (4 + 4 + 2 + 2)     # residual in / out, one term, next input
+    row["prep_bytes"] = n * (2 * H * D + 3 * G * D) * 2            # q in / out, k in, key and value rows out
+    del runner, sched, model
+    torch.cuda.empty_cache()
+    return row
+
+
 def bench_llama_like(name, s, steps, warmup, device="cuda"):
     """The package's Llama-family stack (B200DecoderLayer: fused RMSNorm, rotary + KV write, paged
     attention, gated silu MLP) at the same width, heads, head size 128, layers, GQA 4:1, bf16."""
@@ -692,11 +808,13 @@ def bench_llama_like(name, s, steps, warmup, device="cuda"):
 def run(steps: int, warmup: int, sizes=None):
     rows = []
     every = list(SIZES.items()) + list(DOZETAR_SIZES.items()) + list(KULESUN_SIZES.items()) + list(KISILIX_SIZES.items()) + \
-        list(LUZOSUN_SIZES.items())
+        list(LUZOSUN_SIZES.items()) + list(SAPIVIK_SIZES.items())
     for name, s in every:
         if sizes and name not in sizes:
             continue
-        if name in LUZOSUN_SIZES:
+        if name in SAPIVIK_SIZES:
+            fns = (bench_sapivik, bench_llama_like) if s["dense"] else (bench_sapivik, bench_dozetar, bench_llama_like)
+        elif name in LUZOSUN_SIZES:
             fns = (bench_luzosun, bench_kulesun, bench_llama_like)
         elif name in KISILIX_SIZES:
             fns = (bench_kisilix, bench_dozetar, bench_llama_like)
