@@ -4,6 +4,8 @@ kernels, so the outputs must agree within the decode parity tolerance (max-abs 3
 on two calls in a row with different shapes (the second call finds the first call's partials in the
 shared scratch) and on the single-split path; requests beyond the 8 MiB scratch must be rejected.
 Collected last on purpose (file name): a failure here must not hide other tests under `pytest -x`."""
+import gc
+
 import pytest
 import torch
 
@@ -51,6 +53,7 @@ def _run_both(c, splits):
     _lib.check(lib.b200_attn_decode(*_args(c, o_ref), ws.data_ptr(), ws.numel(), splits, stream),
                "b200_attn_decode")
     torch.cuda.synchronize()
+    gc.collect()                # tensors in reference cycles of earlier tests must not go away in between
     before = torch.cuda.memory_allocated()
     _lib.check(lib.b200_attn_decode_noalloc(*_args(c, o_new), splits, stream), "b200_attn_decode_noalloc")
     torch.cuda.synchronize()
