@@ -900,7 +900,7 @@ int b200_diff_attn_extend(const void* q, int64_t q_stride, const void* pool, int
                           float out_mult, float eps, int dtype, void* stream);
 
 /* ---- channel-gated memories, tied keys and values, identity experts, looped stacks -----------------
- * b200_linear_recurrence with a forget gate per key channel that also decides what is written:
+ * b200_linear_recurrence with a forget gate per key channel that doubles as the write gate:
  * w = (1 - f_lower) * sigmoid(-(zf + f_bias)), S <- S + w (v - S) per channel row, o = S^T q.  zf [T, H * D]
  * pre-activations in the model dtype, f_bias / f_lower fp32 [H * D] (NULL: zero), act 1: silu on q.
  * State rows as the decay form's (b200_linear_recurrence_state_width(..., 0)).                      */

@@ -1,7 +1,7 @@
 """Configuration of the Sapivik design: a decoder-only model over a 32-bit residual with an RMS norm on both
 sides of every sublayer and a residual multiplier,
 
-    x <- x + m norm1b(mixer(norm1(x))),     x <- x + m norm2b(ff(norm2(x))),
+    x += m * post_1(mixer(pre_1(x)))        x += m * post_2(ff(pre_2(x)))
 
 whose mixers are channel-gated matrix memories ("hgrn2") or grouped-query attention with tied keys and values
 ("attention"), whose feed-forwards are clamped gated MLPs ("dense"), mixtures with identity experts and a

@@ -1,5 +1,4 @@
-// The channel-gated memory of linear_recurrence.cu (S_t = diag(f_t) S_(t-1) + w_t v_t^T, w = 1 - f,
-// o_t = S_t^T q_t) for long prompt portions, 16 tokens at a time.  Within a chunk that starts from S_0, with
+// The channel-gated memory of linear_recurrence.cu (S <- diag(f) S + w v^T, w = 1 - f, then o = S^T q) for long prompt portions, 16 tokens at a time.  Within a chunk that starts from S_0, with
 // f_(a,b] = prod_{a < s <= b} f_s per channel:
 //
 //   o_i  = (q_i f_(0,i])^T S_0 + sum_{j <= i} A_ij v_j,      A_ij = sum_d q_i[d] w_j[d] f_(j,i][d]

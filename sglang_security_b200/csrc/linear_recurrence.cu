@@ -10,7 +10,7 @@
 //             value column that is always 1.  The kernel returns the un-normalised o_t together with
 //             n_t . q_t and m_t per (token, head); the consumer divides by
 //             max(|n_t . q_t|, exp(-m_t)) + den_eps                                          (mLSTM)
-//   channel form : a forget gate per key channel that also decides what is written (HGRN2): with
+//   channel form : a forget gate per key channel that doubles as the write gate (HGRN2): with
 //             w = (1 - lower) * sigmoid(-(zf + bias)) per head and channel,
 //             S_t = diag(1 - w_t) S_(t-1) + w_t v_t^T, computed as S += w (v - S): the share that is
 //             forgotten is the share that is written, so the two can not drift apart by rounding; the share w

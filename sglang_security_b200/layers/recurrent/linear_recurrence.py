@@ -13,10 +13,10 @@ the sequence was cut.  Two mixers are built on it:
                             a weight over all heads, an output gate sigmoid(W_g h), W_o
     DecayedLinearAttention  constant decay per head, silu on q, k and v, RMS norm over all heads
                             together with a weight, an output gate, W_o
-    ChannelForgetMixer      a forget gate per head and channel between a lower bound and 1 that also decides
-                            what is written (Qin et al., "HGRN2: Gated Linear RNNs with State Expansion"):
-                            f = l + (1 - l) sigmoid(W_f h + b), S = diag(f) S + (1 - f) v^T, o = S^T silu(W_q h),
-                            RMS norm per head with one weight shared by the heads, W_o
+    ChannelForgetMixer      one gate per channel for forgetting and writing (Qin et al., "HGRN2: Gated Linear
+                            RNNs with State Expansion"): share w = (1 - lower) sigmoid(-(z + bias)),
+                            S += w (v - S) per channel row, o = S^T silu(q), RMS norm of every head with a
+                            weight all heads use, W_o
 """
 from __future__ import annotations
 

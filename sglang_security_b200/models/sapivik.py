@@ -1,13 +1,13 @@
 """Sapivik: decoder-only model over a 32-bit residual stream with an RMS norm on both sides of every sublayer,
-in which a range of layers runs several times in a row with the same weights:
+in which a range of layers is repeated, each pass with the weights of the first:
 
     x = embed[token]
-    per layer run:  x += m norm_1b(mixer(norm_1(x)))
-                    x += m norm_2b(ff(norm_2(x)))              (layers with a feed-forward)
+    per layer run:  x += m * post_1(mixer(pre_1(x)))
+                    x += m * post_2(ff(pre_2(x)))              (layers with a feed-forward)
     ahead of every pass of the loop but the first:  x += embed[token]
     logits = head(norm_f(x))
 
-A layer's mixer is a matrix memory with a forget gate per head and channel ("hgrn2") or grouped-query
+A layer's mixer is a matrix memory gated channel by channel ("hgrn2") or grouped-query
 attention whose values are the projected keys, with unit-norm rotated queries and keys, capped scores and an
 element-wise output gate ("attention").  The feed-forward is a clamped gated MLP or a mixture of silu-gated
 experts, some of which return their input, with a gated shared expert.  Norms, gates and memories, angles,
