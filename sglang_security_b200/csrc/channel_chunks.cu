@@ -1,5 +1,6 @@
-// The channel-gated memory of linear_recurrence.cu (S <- diag(f) S + w v^T, w = 1 - f, then o = S^T q) for long prompt portions, 16 tokens at a time.  Within a chunk that starts from S_0, with
-// f_(a,b] = prod_{a < s <= b} f_s per channel:
+// The channel-gated memory of linear_recurrence.cu (S <- diag(f) S + w v^T, w = 1 - f, then o = S^T q) for long
+// prompt portions, 16 tokens at a time.  Within a chunk that starts from S_0, with f_(a,b] = prod_{a < s <= b} f_s
+// per channel:
 //
 //   o_i  = (q_i f_(0,i])^T S_0 + sum_{j <= i} A_ij v_j,      A_ij = sum_d q_i[d] w_j[d] f_(j,i][d]
 //   S_16 = diag(f_(0,16]) S_0 + sum_j (w_j f_(j,16]) v_j^T
