@@ -282,8 +282,9 @@ __device__ __noinline__ void decode_fused_tail(const TailDev p, int b, int hq0, 
 #include "attn_decode_fp8.cuh"
 namespace b200 {
 
-// HI: the tile holds more than 8 heads (rows 8..15 of the MMA are live).
-template <typename T, int D, int NT, int STAGES, int NW, bool HI, bool TAIL>
+// HI: the tile holds more than 8 heads (rows 8..15 of the MMA are live).  ROWS: the row list and the output gate
+// of b200_attn_decode_rows (an instance of its own: the others stay at their register limit without spills).
+template <typename T, int D, int NT, int STAGES, int NW, bool HI, bool TAIL, bool ROWS = false>
 __global__ void __launch_bounds__(NW * 32, TAIL ? 4 : 0)
 attn_decode_mma_kernel(const DecodeParams p) {
   using C = MmaCfg<D, NT, STAGES, NW>;
@@ -322,7 +323,7 @@ attn_decode_mma_kernel(const DecodeParams p) {
   uint32_t qa[KS][4];
   {
     const int r_lo = lane >> 2, r_hi = r_lo + 8;
-    const T* qb = static_cast<const T*>(p.q) + (p.row_list ? p.row_list[b] : b) * p.q_stride +
+    const T* qb = static_cast<const T*>(p.q) + static_cast<int64_t>(ROWS && p.row_list ? p.row_list[b] : b) * p.q_stride +
                   static_cast<int64_t>(kvh * p.group + head0) * D + (lane & 3) * 2;
     const bool v_lo = r_lo < heads_here, v_hi = HI && r_hi < heads_here;
 #pragma unroll
@@ -550,8 +551,8 @@ attn_decode_mma_kernel(const DecodeParams p) {
     float out = num / den;
     const int hq = kvh * p.group + head0 + h;
     if (p.num_splits == 1) {
-      const int64_t row = p.row_list ? p.row_list[b] : b;
-      if (p.gate) out *= sigmoid_f(to_float<T>(static_cast<const T*>(p.gate)[row * p.gate_stride + hq * D + d]));
+      const int64_t row = ROWS && p.row_list ? p.row_list[b] : b;
+      if (ROWS && p.gate) out *= sigmoid_f(to_float<T>(static_cast<const T*>(p.gate)[row * p.gate_stride + hq * D + d]));
       static_cast<T*>(p.o)[row * p.o_stride + hq * D + d] = from_float<T>(out);
     } else {
       const int64_t pidx = (static_cast<int64_t>(b) * p.Hq + hq) * p.num_splits + split;
@@ -769,6 +770,9 @@ static int launch_decode(const DecodeParams& p, cudaStream_t st) {
   using C = MmaCfg<D, kNT, kStages, kNW>;
   if (p.tickets) return launch_decode_any<C>(attn_decode_mma_kernel<T, D, kNT, kStages, kNW, HI, true>, p, st,
                                              "attn_decode_split", "attn_decode_mma_kernel");
+  if (p.row_list || p.gate)
+    return launch_decode_any<C>(attn_decode_mma_kernel<T, D, kNT, kStages, kNW, HI, false, true>, p, st,
+                                "attn_decode_split", "attn_decode_mma_kernel");
   auto kern = attn_decode_mma_kernel<T, D, kNT, kStages, kNW, HI, false>;
   static bool attr_done = false;
   if (!attr_done) {
